@@ -106,7 +106,7 @@ template <> struct Unpack<__half> {
 };
 
 // dot of two 16B packets accumulated into fp32.
-// half: mixed-precision fma.rn.f32.f16 (SASS FHFMA) -> products are exact in fp32,
+// half: mixed-precision fma.rn.f32.f16 -> products are exact in fp32,
 // bit-identical to convert-then-FFMA but without the conversions.
 __device__ __forceinline__ float fma_h(uint16_t a, uint16_t b, float c) {
 #ifdef B200_NO_FHFMA
@@ -204,7 +204,7 @@ __device__ __forceinline__ void pdl_launch_dependents() {
 }
 
 // ---------------------------------------------------------------------------
-// mbarrier + 1-D bulk async copy (TMA engine, SASS UBLKCP)
+// mbarrier + 1-D bulk async copy (TMA engine)
 // ---------------------------------------------------------------------------
 __device__ __forceinline__ uint32_t smem_u32(const void* p) {
     return (uint32_t)__cvta_generic_to_shared(p);

@@ -10,7 +10,7 @@
 // separately, every phase pays launch + ramp + tail and the weight prefetch of the next kernel is
 // capped by what two co-resident CTAs can hold. Here one CTA per SM stays resident (cooperative
 // launch), a producer warp streams the WHOLE step's weights through one deep smem ring with 1-D
-// bulk copies (cp.async.bulk, UBLKCP) and never waits for a phase boundary, and the 8 consumer
+// bulk copies (cp.async.bulk) and never waits for a phase boundary, and the 8 consumer
 // warps walk a small program of ops separated by grid barriers; while consumers wait at a
 // barrier the ring (up to ~190 KB per SM, ~28 MB chip-wide) keeps HBM busy.
 //
@@ -980,7 +980,7 @@ __device__ __noinline__ void attn_consume(const StepOp& op, const StepParams& p,
         }
 
         // G = 4 / 8 (8 = the 70B-shaped tensor-parallel ranks): eight heads' q, (m, l) and 64 fp32 outputs per lane do not fit
-        // the 168-register cap (G = 8: 472 bytes of stack, 319 local loads / stores in the SASS; G = 4: 136 / 106). A work item
+        // the 168-register cap (ptxas -v reports 472 bytes of stack at G = 8, 136 at G = 4). A work item
         // therefore covers GC = 2 query heads of its (sequence, kv head, split); the NP = G / GC head groups are separate items
         // that other CTAs take (each re-reads the split's K / V rows, from L2 after the first: a few hundred KB per layer
         // against ~100 MB of weights). Per-head arithmetic and its order are unchanged. Measured on an 8-layer 70B-shaped

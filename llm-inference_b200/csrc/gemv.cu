@@ -8,11 +8,11 @@
 // Structure (HBM-bound; algorithmic bytes = N*K*sizeof(T) + small vectors):
 //  * one persistent CTA per SM owns a contiguous, byte-balanced range of row-pair "units";
 //  * a producer warp streams those rows through a ring of 32 KB stages with 1-D bulk async
-//    copies (cp.async.bulk -> SASS UBLKCP, completion on an mbarrier); each stage holds
+//    copies (cp.async.bulk, completion on an mbarrier); each stage holds
 //    8 units x 2 rows x 2 KB K-segment;
 //  * 8 consumer warps: warp w owns unit w of the stage, dots both rows against x held in
 //    shared memory (one x packet read serves two weight packets), fp32 accumulation
-//    (fma.rn.f32.f16 -> FHFMA for half), warp-shuffle reduce at the end of the row;
+//    (fma.rn.f32.f16 for half), warp-shuffle reduce at the end of the row;
 //    from 2 fp16 token rows on the consumers switch to mma.sync (kSegPitchMma below): measured at batch 2 / 3 / 4,
 //    7B shapes, fused order, context 512: 3.50 / 4.45 / 4.71 -> 3.39 / 3.82 / 4.07 ms per step;
 //  * under programmatic dependent launch the producer starts streaming WEIGHTS before
