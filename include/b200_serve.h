@@ -12,7 +12,9 @@
  * frequency interpolation; dense or routed squared-relu feed-forwards; a repeated span of layers), "Sakevik" (norms on the
  * sublayers' outputs; a hashed pair embedding; layers of an element-wise gated recurrence, of windowed attention with sigmoid
  * weights, rotated values and head gates, or of windowed latent attention with a shared rotary key part; clamped gated
- * feed-forwards), "llama" (the reference's weight directory, llama_weights.cc:41-53, with
+ * feed-forwards), "Filipel" (parallel layers of latent attention with low-rank queries, or of windowed attention whose weights
+ * are mixed across heads beside a state-space recurrence; routed experts in groups, a dense feed-forward of normed powers),
+ * "llama" (the reference's weight directory, llama_weights.cc:41-53, with
  * a config.json naming the b200_model_config fields).
  */
 #ifndef B200_SERVE_H
@@ -38,7 +40,7 @@ int b200_embed_positions(const int* ids, const int* pos, const void* table, cons
 
 /* Layer norm with weight and bias, up to two (w, b) pairs applied to the SAME rows of x (mean and variance are
  * computed once, two-pass, in fp32): out_k[i,:] = (x[r_i,:] - mean) / sqrt(var + eps) * w_k + b_k, r_i = rows ? rows[i]
- * : i. x fp32 [*, width]; w, b fp32; out1 / out2 of out_dtype (out2, w2, b2 may be NULL). */
+ * : i. x fp32 [*, width]; w, b fp32; out1 / out2 of out_dtype (out2, w2 may be NULL; b1, b2 NULL: no bias). */
 int b200_layernorm_pair(const float* x, const int* rows, int n_rows, int width, float eps, const float* w1,
                         const float* b1, void* out1, const float* w2, const float* b2, void* out2, int out_dtype,
                         void* stream);
@@ -125,6 +127,18 @@ int b200_latent_attention_ex(const b200_latent_attention_args* a, void* stream);
 int b200_latent_store_rot(const float* raw, long long ld_raw, const float* w, float eps, void* pool, const int* pages,
                           int max_pages, int page_rows, const int* slot, const int* pos, int n_tokens, int rank, int extra,
                           const float* cos, const float* sin, int rot_layout, int dtype, void* stream);
+/* The two low-rank rows that a latent layer norms before anything else reads them, one launch: q_out[t, 0:q_rank] =
+ * norm(raw[t, q_off : q_off + q_rank]) * q_norm as `dtype` (the operand of the query up-projection), and, when pool is not NULL,
+ * the cache row of b200_latent_store_rot from raw[t, kv_off : kv_off + rank + extra]. */
+typedef struct b200_latent_norms_args {
+    const float* raw; long long ld_raw; int q_off, kv_off;
+    const float* q_norm; int q_rank; void* q_out;
+    const float* kv_norm; float eps; void* pool;
+    const int* pages; int max_pages, page_rows; const int* slot; const int* pos;
+    int n_tokens, rank, extra;
+    const float* cos; const float* sin; int rot_layout, dtype;
+} b200_latent_norms_args;
+int b200_latent_norms(const b200_latent_norms_args* a, void* stream);
 /* dst[t, h, dst_off + i] = rot(src[t, src_off + h * src_stride + 0:dims])[i] for i < dims: the rotated part of every head's
  * query placed behind its absorbed part (fp32 to fp32; dst rows of ld_dst floats, heads dst_stride apart) */
 int b200_rotate_part(const float* src, long long ld_src, long long src_off, long long src_stride, float* dst, long long ld_dst,
@@ -140,6 +154,12 @@ int b200_moe_route(const void* h, int h_dtype, const float* w_router, const floa
  * chosen (ties: the lower index) and their weights are the softmax over the chosen logits only. */
 int b200_moe_route_logits(const void* h, int h_dtype, const float* w_router, const float* bias, int n_tokens, int width,
                           int n_out, int top, int* chosen, float* weight, void* stream);
+/* Router with groups of neighbouring experts: s = softmax(h W_r^T) over all n_out outputs (fp32 accumulate); a group's score is
+ * the largest s in it and only experts of the best `keep` of `groups` equal groups can be chosen; the `top` largest s among
+ * them are (ties: the lower index, for groups and experts); weights are s / (sum of the chosen s + 1e-20).
+ * n_out must be a multiple of groups and top at most keep * n_out / groups. groups 1: no restriction. */
+int b200_moe_route_groups(const void* h, int h_dtype, const float* w_router, int n_tokens, int width, int n_out, int top,
+                          int groups, int keep, int* chosen, float* weight, void* stream);
 /* Counting sort of the (token, choice) pairs by expert: group_off [n_experts + 1], src_row [n_tokens * top] (token of
  * each sorted row), dest [n_tokens, top] (sorted row of each pair, -1 for chosen >= n_experts: identity experts own no
  * rows). One launch, no host sync. */
@@ -188,6 +208,28 @@ typedef struct b200_rmsnorm_residual_args {
     int norm_addend; const float* y_bias;
 } b200_rmsnorm_residual_args;
 int b200_rmsnorm_residual(const b200_rmsnorm_residual_args* a, void* stream);
+
+/* Residual update of a parallel layer (every sublayer reads the same normed row) fused with the layer norm that reads the
+ * residual next, one launch per layer:
+ *   x[t,:] += mult * (s1 * f1(y1[t,:]) + s2 * f2(y2[t,:]) + y3[t,:] + sum_k weight[t,k] * expert_out[dest[t,k],:])
+ *   out[t,:] = (x[t,:] - mean) / sqrt(var + eps) * ln_w + ln_b        (as out_dtype; skipped when ln_w is NULL)
+ * f_i is the identity where w_i is NULL, else v / sqrt(mean(v^2) + eps) * w_i. Every addend may be NULL, ln_b too (fp32 sums in
+ * this fixed order; mean and variance two-pass). */
+typedef struct b200_parallel_residual_args {
+    float* x; float mult;
+    const float* y1; const float* w1; float s1;
+    const float* y2; const float* w2; float s2;
+    const float* y3;
+    const float* expert_out; const int* dest; const float* weight; int top;
+    const float* ln_w; const float* ln_b; float eps;
+    void* out; int out_dtype;
+    int n_rows, width;
+} b200_parallel_residual_args;
+int b200_parallel_residual(const b200_parallel_residual_args* a, void* stream);
+
+/* Dense feed-forward activation of normed powers: out[t,:] = c[0] N(z) + c[1] N(z^2) + c[2] N(z^3) + c[3], z = z[t,:] (fp32
+ * [n_rows, width]), powers element by element, N v = v / sqrt(mean(v^2) + eps) over the row; out of out_dtype. */
+int b200_poly_norm(const float* z, const float* c4, float eps, void* out, int n_rows, int width, int out_dtype, void* stream);
 
 /* Rotary positions: cos_out / sin_out [n_tokens, n_freq] = cos / sin(pos[t] * freq[i]); the angle is formed and reduced in
  * double precision (freq is a device array of doubles, whatever scaling of the frequencies already applied by the
@@ -265,8 +307,18 @@ typedef struct b200_paged_attention_args {
        sigmoid_weights != 0: no softmax; the weight of a visible key is sigmoid(s_j + head_bias[h]) (head_bias fp32 [heads]
        or NULL), not normalised over the keys: out = sum_j w_j v_j. Not with softcap, denom_bias or maps > 1. */
     int window, sigmoid_weights; const float* head_bias;
+    /* head_temp (fp32 [heads] or NULL): the scores of head h are multiplied by head_temp[h] beside `scale`.
+       head_mix (fp32 [heads, heads] or NULL): the normalised softmax weights are mixed across the heads before they meet the
+       values, w_h(j) <- sum_g head_mix[h, g] w_g(j), and head h weights the values of its own key head. Plain softmax only
+       (no softcap, denom_bias, sigmoid_weights, maps > 1). bfloat16 prompt portions run as three tile launches per block of
+       rows (scores and their row statistics; the mix; the weighted values) through the workspace, which
+       b200_mixed_attention_workspace_bytes sizes; single tokens, fp32 and calls without workspace run on a kernel whose CTA
+       (or cluster of CTAs, sharing the context) holds all heads of a token. */
+    const float* head_temp; const float* head_mix;
 } b200_paged_attention_args;
 size_t b200_paged_attention_workspace_bytes(int n_tokens, int heads, int vdim);
+/* longest_seen: most keys a token sees before the window is applied (the longest sequence); window 0: none */
+size_t b200_mixed_attention_workspace_bytes(int n_tokens, int heads, int window, int longest_seen);
 int b200_paged_attention(const b200_paged_attention_args* a, void* stream);
 
 /* Retention: linear attention with a fixed decay per head and a carried state, no softmax. For every entry (a run of
@@ -371,6 +423,33 @@ typedef struct b200_selective_scan_args {
 } b200_selective_scan_args;
 size_t b200_selective_scan_workspace_bytes(int n_tokens, int n_entries, int channels, int n_state);
 int b200_selective_scan(const b200_selective_scan_args* a, void* stream);
+
+/* State-space recurrence with ONE decay per head (a matrix state of n_state x vdim per head, input-dependent step sizes). Per
+ * entry (a run of consecutive tokens of one sequence) and head h (group g = h / (heads / groups)), with
+ * dt = softplus(dt_raw[t, h] + dt_bias[h]):
+ *   S <- exp(dt * A[h]) * S + dt * B[t, g] x[t, h]^T,   out[t, h, :] = S^T C[t, g] + D[h] * x[t, h, :]
+ * x, B, C are columns of one fp32 row: u[t, x_off + h * vdim + :], u[t, b_off + g * n_state + :], u[t, c_off + g * n_state + :]
+ * (leading dimension ld_u); dt_raw fp32 with leading dimension ld_dt; A (already negative), dt_bias, D fp32 [heads]; S fp32
+ * [n_slots, heads, n_state, vdim], starting from zero when the entry starts at position 0 and left in place for the next
+ * step. out fp32 [n_tokens, heads * vdim].
+ * Entries walk token by token in fp32; with chunked != 0, a workspace and an entry of 128 tokens or more, the step takes the
+ * chunk form instead (64-token chunks on tf32 tensor-core products with fp32 accumulation; decays, step sizes, chunk states
+ * and the sums between chunks stay fp32, the decay exponents are summed in double). */
+typedef struct b200_ssd_scan_args {
+    const float* u; long long ld_u; int x_off, b_off, c_off;
+    const float* dt_raw; long long ld_dt; const float* dt_bias;
+    const float* A; const float* D;
+    float* state; float* out;
+    const int* ent_row; const int* ent_len; const int* slot; const int* pos;
+    int n_entries, n_tokens, heads, groups, vdim, n_state, longest_entry, chunked;
+    void* workspace; size_t workspace_bytes;
+} b200_ssd_scan_args;
+size_t b200_ssd_scan_workspace_bytes(int n_tokens, int n_entries, int heads, int groups, int vdim, int n_state);
+int b200_ssd_scan(const b200_ssd_scan_args* a, void* stream);
+/* out[t, c] = v / sqrt(mean over v's part + eps) * w[c], v = y[t, c] * silu(z[t, c]); the row of n columns is normed in `parts`
+ * equal parts. y fp32 [n_tokens, n], z fp32 with leading dimension ld_z, w fp32 [n]; out of out_dtype. */
+int b200_gated_group_rms(const float* y, const float* z, long long ld_z, const float* w, void* out, int n_tokens, int n, int parts,
+                         float eps, int out_dtype, void* stream);
 
 /* ---------------------------------------------------------------------------------------------
  * models

@@ -8,6 +8,9 @@
 // score plus a number per head instead of a softmax: then nothing is normalised over the keys, which in the running
 // (maximum, denominator, output) form is a maximum held at 0 and a denominator held at 1.
 //
+// Scores can carry a factor per head; weights that are mixed across heads before they meet the values are the business of
+// mixed_attention.cu.
+//
 //   paged_attn_row_kernel   one CTA per (token, query head), fp32 arithmetic on caches of either dtype: each warp
 //                           takes blocks of 32 keys (a lane scores one key; the weighted value sum runs with a lane per
 //                           output column), keeps its own running maximum / denominator / output and the warps merge at
@@ -22,31 +25,11 @@
 #include "b200_serve.h"
 #include "common.cuh"
 #include "launch_count.h"
+#include "paged_attention.cuh"
 
 namespace b200 {
 
-struct PA {
-    const void* q; void* out; const void* k_pool; const void* v_pool;
-    const int* pages; int max_pages, page_rows;
-    const int* slot; const int* pos;
-    int n_tokens, heads, kv_heads, dim, vdim;
-    float scale, softcap, denom_bias;
-    int splits; float* part;   // row kernel: shares of a context split over gridDim.z CTAs, [token, head, split, 2 + vdim]
-    int chunk, maps, out_f32;
-    int window, sigmoid; const float* head_bias;
-};
-// first key that position p sees
-__device__ __forceinline__ int pa_first_key(const PA& a, int p) {
-    const int f = a.chunk > 0 ? (p / a.chunk) * a.chunk : 0;
-    return a.window > 0 ? max(f, p - a.window + 1) : f;
-}
 __device__ __forceinline__ float pa_sigmoid(float v) { return 1.f / (1.f + expf(-v)); }
-template <typename T>
-__device__ __forceinline__ void pa_store(const PA& a, size_t idx, float v) {
-    if (a.out_f32) reinterpret_cast<float*>(a.out)[idx] = v;
-    else reinterpret_cast<T*>(a.out)[idx] = DT<T>::from_f(v);
-}
-
 constexpr int kRowWarps = 4;
 constexpr int kMaxSplits = 16;
 constexpr int kMaxVPerLane = 8;   // vdim <= 256
@@ -102,7 +85,7 @@ __global__ void __launch_bounds__(kRowWarps * 32) paged_attn_row_kernel(const PA
     const int per = ((p - j_lo + a.splits) / a.splits + 31) & ~31;
     const int j_begin = j_lo + blockIdx.z * per, j_end = min(p + 1, j_begin + per);
     if (warp == 0 && blockIdx.z == 0 && a.denom_bias > 0.f) { m = 0.f; l = a.denom_bias; }
-    const float hb = (a.sigmoid && a.head_bias) ? a.head_bias[h / a.maps] : 0.f;
+    const float hb = (a.sigmoid && a.head_bias) ? a.head_bias[h / a.maps] : 0.f, sc_h = pa_scale(a, h / a.maps);
     if (a.sigmoid) { m = 0.f; l = (warp == 0 && blockIdx.z == 0) ? 1.f : 0.f; }
     for (int j0 = j_begin + warp * 32; j0 < j_end; j0 += kRowWarps * 32) {
         const int j = j0 + lane;
@@ -111,7 +94,7 @@ __global__ void __launch_bounds__(kRowWarps * 32) paged_attn_row_kernel(const PA
         float s = -INFINITY;
         if (ok) {
             row = (size_t)plist[j / a.page_rows] * a.page_rows + j % a.page_rows;
-            s = dot_row<T>(qs, K + (row * k_units + ku) * a.dim, a.dim) * a.scale;
+            s = dot_row<T>(qs, K + (row * k_units + ku) * a.dim, a.dim) * sc_h;
             if (a.softcap > 0.f) s = a.softcap * tanhf(s / a.softcap);
         }
         float bm = s;
@@ -168,14 +151,6 @@ __global__ void __launch_bounds__(kRowWarps * 32) paged_attn_row_kernel(const PA
 // the group from one pass over the keys and values. Eight lanes share a key row (16-byte loads, a row is read once,
 // whole sectors), four keys per warp step; the scores of 32 keys go through shared memory to the softmax (a lane per
 // key) and on to the weighted value sum (a lane per pair of output columns). fp32 arithmetic on caches of either dtype.
-template <typename T> struct Pair;
-template <> struct Pair<float> {
-    static __device__ __forceinline__ float2 load(const float* p) { return *reinterpret_cast<const float2*>(p); }
-};
-template <> struct Pair<__nv_bfloat16> {
-    static __device__ __forceinline__ float2 load(const __nv_bfloat16* p) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p)); }
-};
-
 template <typename T, int R>   // R query heads per key head
 __global__ void __launch_bounds__(kRowWarps * 32) paged_attn_group_kernel(const PA a) {
     extern __shared__ float sm[];
@@ -252,7 +227,7 @@ __global__ void __launch_bounds__(kRowWarps * 32) paged_attn_group_kernel(const 
                 rows[warp][kk] = row;
 #pragma unroll
                 for (int r = 0; r < R; ++r) {
-                    float sv = acc[r] * a.scale;
+                    float sv = acc[r] * pa_scale(a, g * R + r);
                     if (a.softcap > 0.f) sv = a.softcap * tanhf(sv / a.softcap);
                     scw[r * 32 + kk] = j < j_end ? sv : -INFINITY;
                 }
@@ -371,25 +346,6 @@ __global__ void __launch_bounds__(128) paged_attn_combine_kernel(const float* __
 // ---------------------------------------------------------------------------------------------------------------
 constexpr int kTileM = 64, kTileN = 64;
 
-__device__ __forceinline__ void pa_ldsm_x4(uint32_t (&r)[4], const void* p) {
-    const uint32_t a = (uint32_t)__cvta_generic_to_shared(p);
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
-}
-__device__ __forceinline__ void pa_ldsm_x4_trans(uint32_t (&r)[4], const void* p) {
-    const uint32_t a = (uint32_t)__cvta_generic_to_shared(p);
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
-}
-// (not volatile: a pure function of its registers, so the compiler may interleave independent accumulators)
-__device__ __forceinline__ void pa_mma(float (&d)[4], const uint32_t (&a)[4], const uint32_t (&b)[2]) {
-    asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b[0]), "r"(b[1]));
-}
-__device__ __forceinline__ uint32_t pa_pack(float lo, float hi) {
-    const __nv_bfloat162 h = __floats2bfloat162_rn(lo, hi);
-    return *reinterpret_cast<const uint32_t*>(&h);
-}
-
 template <int D, int DV, bool BLOCKS>   // dim == D (a multiple of 32), vdim == DV (a multiple of 16); BLOCKS: a block mask or a window
 __global__ void __launch_bounds__(128, DV <= 128 ? 3 : 2) paged_attn_tile_kernel(const PA a) {
     using bf = __nv_bfloat16;
@@ -433,7 +389,7 @@ __global__ void __launch_bounds__(128, DV <= 128 ? 3 : 2) paged_attn_tile_kernel
     float m_run[2] = {m0, m0}, l_run[2] = {l0, l0};
     const float hb = (sig && a.head_bias) ? a.head_bias[h / a.maps] : 0.f;
     const int r_lo = warp * 16 + gid, r_hi = r_lo + 8;
-    const float scale_over_cap = a.softcap > 0.f ? a.scale / a.softcap : 0.f;
+    const float sc_h = pa_scale(a, h / a.maps), scale_over_cap = a.softcap > 0.f ? sc_h / a.softcap : 0.f;
     const bf* Kp = reinterpret_cast<const bf*>(a.k_pool);
     const bf* Vp = reinterpret_cast<const bf*>(a.v_pool);
 
@@ -532,7 +488,7 @@ __global__ void __launch_bounds__(128, DV <= 128 ? 3 : 2) paged_attn_tile_kernel
 #pragma unroll
                 for (int nt = 0; nt < kTileN / 8; ++nt)
 #pragma unroll
-                    for (int e = 0; e < 4; ++e) s[nt][e] *= a.scale;
+                    for (int e = 0; e < 4; ++e) s[nt][e] *= sc_h;
             }
             float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
@@ -655,13 +611,15 @@ extern "C" int b200_paged_attention(const b200_paged_attention_args* p, void* st
         p->chunk < 0 || p->maps < 0 || p->window < 0)
         return B200_EINVAL;
     if (p->sigmoid_weights && (p->softcap > 0.f || p->denom_bias > 0.f || p->maps > 1)) return B200_EINVAL;
+    if (p->head_mix && (p->softcap > 0.f || p->denom_bias > 0.f || p->sigmoid_weights || p->maps > 1)) return B200_EINVAL;
     const int maps = p->maps > 0 ? p->maps : 1, units = p->heads * maps;
-    if (p->vdim > 32 * kMaxVPerLane) return B200_EUNSUPPORTED;
+    if (!p->head_mix && p->vdim > 32 * kMaxVPerLane) return B200_EUNSUPPORTED;
     if (p->n_tokens == 0) return B200_OK;
     PA a{p->q, p->out, p->k_pool, p->v_pool, p->pages, p->max_pages, p->page_rows, p->slot, p->pos, p->n_tokens, p->heads,
          p->kv_heads, p->dim, p->vdim, p->scale, p->softcap, p->denom_bias, 1, nullptr, p->chunk, maps, p->out_f32,
-         p->window, p->sigmoid_weights != 0, p->head_bias};
+         p->window, p->sigmoid_weights != 0, p->head_bias, p->head_temp, p->head_mix};
     cudaStream_t s = (cudaStream_t)stream;
+    if (p->head_mix) return mixed_attention(a, p->dtype, p->longest_entry, p->longest_context, p->workspace, p->workspace_bytes, s);
     const size_t smem = ((size_t)p->dim + (size_t)kRowWarps * p->vdim) * sizeof(float);
     if (smem > 48 * 1024) return B200_EUNSUPPORTED;
     auto al16 = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15u) == 0; };

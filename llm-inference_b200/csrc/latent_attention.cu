@@ -53,23 +53,26 @@ __global__ void __launch_bounds__(128) latent_store_kernel(const float* __restri
     for (int i = threadIdx.x; i < rank; i += blockDim.x) dst[i] = DT<T>::from_f(src[i] * r * w[i]);
 }
 
-// row = [norm(raw[0:rank]) * w | rot(raw[rank:rank+extra])]
-template <typename T>
-__global__ void __launch_bounds__(128) latent_store_rot_kernel(const float* __restrict__ raw, long long ld_raw, const float* __restrict__ w,
-                                                               float eps, T* __restrict__ pool, const int* __restrict__ pages, int max_pages,
-                                                               int page_rows, const int* __restrict__ slot, const int* __restrict__ pos, int rank,
-                                                               int extra, const float* __restrict__ cs, const float* __restrict__ sn, int layout) {
-    __shared__ float red[4];
-    const int t = blockIdx.x;
-    const float* src = raw + (size_t)t * ld_raw;
+// 1 / sqrt(mean(src[0:n]^2) + eps) over a CTA of 128 threads
+__device__ __forceinline__ float row_rinv(const float* src, int n, float eps, float* red) {
     float q = 0.f;
-    for (int i = threadIdx.x; i < rank; i += blockDim.x) q += src[i] * src[i];
+    for (int i = threadIdx.x; i < n; i += blockDim.x) q += src[i] * src[i];
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) q += __shfl_xor_sync(0xffffffffu, q, o);
     if (threadIdx.x % 32 == 0) red[threadIdx.x / 32] = q;
     __syncthreads();
     const float tot = red[0] + red[1] + red[2] + red[3];
-    const float r = 1.0f / sqrtf(tot / (float)rank + eps);
+    return 1.0f / sqrtf(tot / (float)n + eps);
+}
+
+// row = [norm(raw[0:rank]) * w | rot(raw[rank:rank+extra])]
+template <typename T>
+__device__ __forceinline__ void store_rot_row(const float* raw, long long ld_raw, const float* w, float eps, T* pool, const int* pages,
+                                              int max_pages, int page_rows, const int* slot, const int* pos, int rank, int extra,
+                                              const float* cs, const float* sn, int layout, float* red) {
+    const int t = blockIdx.x;
+    const float* src = raw + (size_t)t * ld_raw;
+    const float r = row_rinv(src, rank, eps, red);
     const int p = pos[t];
     const size_t row = (size_t)pages[(size_t)slot[t] * max_pages + p / page_rows] * page_rows + p % page_rows;
     T* dst = pool + row * (rank + extra);
@@ -77,6 +80,29 @@ __global__ void __launch_bounds__(128) latent_store_rot_kernel(const float* __re
     const int nf = extra / 2;
     for (int i = threadIdx.x; i < extra; i += blockDim.x)
         dst[rank + i] = DT<T>::from_f(rotary_component(src + rank, i, 2 * nf, layout, cs + (size_t)t * nf, sn + (size_t)t * nf));
+}
+
+template <typename T>
+__global__ void __launch_bounds__(128) latent_store_rot_kernel(const float* __restrict__ raw, long long ld_raw, const float* __restrict__ w,
+                                                               float eps, T* __restrict__ pool, const int* __restrict__ pages, int max_pages,
+                                                               int page_rows, const int* __restrict__ slot, const int* __restrict__ pos, int rank,
+                                                               int extra, const float* __restrict__ cs, const float* __restrict__ sn, int layout) {
+    __shared__ float red[4];
+    store_rot_row<T>(raw, ld_raw, w, eps, pool, pages, max_pages, page_rows, slot, pos, rank, extra, cs, sn, layout, red);
+}
+
+// blockIdx.y 0: the normed query row as GEMM operand; 1: the cache row
+template <typename T>
+__global__ void __launch_bounds__(128) latent_norms_kernel(const b200_latent_norms_args a) {
+    __shared__ float red[4];
+    if (blockIdx.y == 0) {
+        const float* src = a.raw + (size_t)blockIdx.x * a.ld_raw + a.q_off;
+        const float r = row_rinv(src, a.q_rank, a.eps, red);
+        T* dst = reinterpret_cast<T*>(a.q_out) + (size_t)blockIdx.x * a.q_rank;
+        for (int i = threadIdx.x; i < a.q_rank; i += blockDim.x) dst[i] = DT<T>::from_f(src[i] * r * a.q_norm[i]);
+    } else
+        store_rot_row<T>(a.raw + a.kv_off, a.ld_raw, a.kv_norm, a.eps, reinterpret_cast<T*>(a.pool), a.pages, a.max_pages, a.page_rows, a.slot,
+                         a.pos, a.rank, a.extra, a.cos, a.sin, a.rot_layout, red);
 }
 
 template <typename T>
@@ -461,6 +487,19 @@ extern "C" int b200_latent_store_rot(const float* raw, long long ld_raw, const f
                                                                extra, cos, sin, rot_layout);
     else
         return B200_EINVAL;
+    count_launch();
+    return (int)cudaGetLastError();
+}
+
+extern "C" int b200_latent_norms(const b200_latent_norms_args* a, void* stream) {
+    if (!a || !a->raw || !a->q_norm || !a->q_out || a->q_rank < 1 || a->n_tokens < 0 || a->q_off < 0) return B200_EINVAL;
+    if (a->pool && (!a->kv_norm || !a->pages || !a->slot || !a->pos || a->rank < 1 || a->extra < 0 || a->page_rows < 1 || a->kv_off < 0)) return B200_EINVAL;
+    if (a->pool && a->extra > 0 && (!a->cos || !a->sin || (a->rot_layout != B200_ROPE_HALF && a->rot_layout != B200_ROPE_INTERLEAVED))) return B200_EINVAL;
+    if (a->n_tokens == 0) return B200_OK;
+    const dim3 grid(a->n_tokens, a->pool ? 2 : 1);
+    if (a->dtype == B200_BF16) latent_norms_kernel<__nv_bfloat16><<<grid, 128, 0, (cudaStream_t)stream>>>(*a);
+    else if (a->dtype == B200_F32) latent_norms_kernel<float><<<grid, 128, 0, (cudaStream_t)stream>>>(*a);
+    else return B200_EINVAL;
     count_launch();
     return (int)cudaGetLastError();
 }

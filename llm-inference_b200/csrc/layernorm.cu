@@ -58,8 +58,8 @@ __global__ void __launch_bounds__(256) layernorm_pair_kernel(const float* __rest
     const float rstd = 1.0f / sqrtf(ln_block_sum(q, red) / (float)width + eps);
     for (int c = threadIdx.x; c < width; c += blockDim.x) {
         const float n = (row[c] - mean) * rstd;
-        out1[(size_t)i * width + c] = DT<T>::from_f(n * w1[c] + b1[c]);
-        if (out2) out2[(size_t)i * width + c] = DT<T>::from_f(n * w2[c] + b2[c]);
+        out1[(size_t)i * width + c] = DT<T>::from_f(n * w1[c] + (b1 ? b1[c] : 0.f));
+        if (out2) out2[(size_t)i * width + c] = DT<T>::from_f(n * w2[c] + (b2 ? b2[c] : 0.f));
     }
 }
 
@@ -351,20 +351,20 @@ extern "C" int b200_embed_positions(const int* ids, const int* pos, const void* 
 extern "C" int b200_layernorm_pair(const float* x, const int* rows, int n_rows, int width, float eps, const float* w1,
                                    const float* b1, void* out1, const float* w2, const float* b2, void* out2, int out_dtype,
                                    void* stream) {
-    if (!x || !w1 || !b1 || !out1 || n_rows < 0 || width < 1) return B200_EINVAL;
-    if (out2 && (!w2 || !b2)) return B200_EINVAL;
+    if (!x || !w1 || !out1 || n_rows < 0 || width < 1) return B200_EINVAL;
+    if (out2 && !w2) return B200_EINVAL;
     if (n_rows == 0) return B200_OK;
     const size_t smem = (size_t)width * sizeof(float);
     if (smem > 200 * 1024) return B200_EUNSUPPORTED;
     cudaStream_t s = (cudaStream_t)stream;
     if (out_dtype == B200_BF16) {
         static unsigned long long done = 0;
-        if (smem > 48 * 1024) ensure_max_dynamic_smem((const void*)layernorm_pair_kernel<__nv_bfloat16>, (int)smem, done);
+        if (smem > 48 * 1024) ensure_max_dynamic_smem((const void*)layernorm_pair_kernel<__nv_bfloat16>, 200 * 1024, done);
         layernorm_pair_kernel<__nv_bfloat16><<<n_rows, 256, smem, s>>>(x, rows, width, eps, w1, b1, (__nv_bfloat16*)out1, w2, b2,
                                                                       (__nv_bfloat16*)out2);
     } else if (out_dtype == B200_F32) {
         static unsigned long long done = 0;
-        if (smem > 48 * 1024) ensure_max_dynamic_smem((const void*)layernorm_pair_kernel<float>, (int)smem, done);
+        if (smem > 48 * 1024) ensure_max_dynamic_smem((const void*)layernorm_pair_kernel<float>, 200 * 1024, done);
         layernorm_pair_kernel<float><<<n_rows, 256, smem, s>>>(x, rows, width, eps, w1, b1, (float*)out1, w2, b2, (float*)out2);
     } else
         return B200_EINVAL;

@@ -145,8 +145,17 @@ int SequenceBatch::release(int slot) {
 StepRunner::~StepRunner() {
     if (stream_) cudaStreamSynchronize(stream_);
     drop_graphs();
+    for (cudaStream_t s : side_) { cudaStreamSynchronize(s); cudaStreamDestroy(s); }
+    for (cudaEvent_t e : side_done_) cudaEventDestroy(e);
+    if (groups_ready_) cudaEventDestroy(groups_ready_);
+    if (group_off_host_) cudaFreeHost(group_off_host_);
+    for (Lane& l : lanes_) {
+        if (l.stream) { cudaStreamSynchronize(l.stream); cudaStreamDestroy(l.stream); }
+        if (l.forked) cudaEventDestroy(l.forked);
+        if (l.joined) cudaEventDestroy(l.joined);
+        cudaFree(l.ws);
+    }
     for (void* p : owned_) cudaFree(p);
-    cudaFree(ws_);
     cudaFree(attn_ws_);
     cudaFree(capture_);
     if (logits_host_) cudaFreeHost(logits_host_);
@@ -155,6 +164,10 @@ StepRunner::~StepRunner() {
 
 int StepRunner::init_runner(std::string& err) {
     if (cudaStreamCreateWithFlags(&stream_, cudaStreamNonBlocking) != cudaSuccess) { err = "no CUDA device: this library has no CPU path"; return B200_EINVAL; }
+    for (int k = 1; k < kLanes; ++k)
+        if (cudaStreamCreateWithFlags(&lanes_[k].stream, cudaStreamNonBlocking) != cudaSuccess ||
+            cudaEventCreateWithFlags(&lanes_[k].forked, cudaEventDisableTiming) != cudaSuccess ||
+            cudaEventCreateWithFlags(&lanes_[k].joined, cudaEventDisableTiming) != cudaSuccess) { err = "streams of the step's lanes"; return B200_EINVAL; }
     const char* e = getenv("B200_NO_GRAPH");
     graphs_enabled_ = !(e && e[0] == '1');
     return B200_OK;
@@ -207,17 +220,81 @@ int StepRunner::ensure_logits_host(int W) {
     return B200_OK;
 }
 
-int StepRunner::gemm(const void* A, const void* W, void* C, int c_dt, int M, int N, int K, int epi, float epi_param) {
+int StepRunner::gemm(const void* A, const void* W, void* C, int c_dt, int M, int N, int K, int epi, float epi_param, int k) {
     const size_t need = b200_linear_ex_workspace_bytes(M, N, K);
-    if (need > ws_bytes_ && !capturing_) {
-        cudaStreamSynchronize(stream_);
+    Lane& l = lanes_[k];
+    if (need > l.ws_bytes && !capturing_) {
+        cudaStreamSynchronize(lane(k));
         ++buffers_epoch_;
-        cudaFree(ws_);
-        ws_ = nullptr;
-        ws_bytes_ = 0;
-        if (cudaMalloc(&ws_, need) == cudaSuccess) ws_bytes_ = need;   // without it the call runs with a single split
+        cudaFree(l.ws);
+        l.ws = nullptr;
+        l.ws_bytes = 0;
+        if (cudaMalloc(&l.ws, need) == cudaSuccess) l.ws_bytes = need;   // without it the call runs with a single split
     }
-    return b200_linear_ex2(A, W, C, M, N, K, dtype_, c_dt, epi, epi_param, ws_, ws_bytes_, stream_);
+    return b200_linear_ex2(A, W, C, M, N, K, dtype_, c_dt, epi, epi_param, l.ws, l.ws_bytes, lane(k));
+}
+
+int StepRunner::fork(int k, std::string& err) {
+    cudaError_t e = cudaEventRecord(lanes_[k].forked, stream_);
+    if (e == cudaSuccess) e = cudaStreamWaitEvent(lanes_[k].stream, lanes_[k].forked, 0);
+    if (e != cudaSuccess) { err = std::string("step: fork: ") + cudaGetErrorString(e); return (int)e; }
+    return B200_OK;
+}
+int StepRunner::join(int k, std::string& err) {
+    cudaError_t e = cudaEventRecord(lanes_[k].joined, lanes_[k].stream);
+    if (e == cudaSuccess) e = cudaStreamWaitEvent(stream_, lanes_[k].joined, 0);
+    if (e != cudaSuccess) { err = std::string("step: join: ") + cudaGetErrorString(e); return (int)e; }
+    return B200_OK;
+}
+
+int StepRunner::expert_rows(const ExpertGroups& g, int k, std::string& err) {
+    if (side_.empty()) {
+        if (cudaEventCreateWithFlags(&groups_ready_, cudaEventDisableTiming) != cudaSuccess) { err = "cudaEventCreate"; return B200_EINVAL; }
+        for (int i = 0; i < kExpertStreams; ++i) {
+            cudaStream_t s = nullptr;
+            cudaEvent_t e = nullptr;
+            if (cudaStreamCreateWithFlags(&s, cudaStreamNonBlocking) != cudaSuccess || cudaEventCreateWithFlags(&e, cudaEventDisableTiming) != cudaSuccess) { err = "cudaStreamCreate"; return B200_EINVAL; }
+            side_.push_back(s);
+            side_done_.push_back(e);
+        }
+    }
+    if (group_off_cap_ < g.experts + 1) {
+        if (group_off_host_) cudaFreeHost(group_off_host_);
+        group_off_host_ = nullptr;
+        group_off_cap_ = 0;
+        if (cudaMallocHost(&group_off_host_, (size_t)(g.experts + 1) * sizeof(int)) != cudaSuccess) { err = "cudaMallocHost"; return B200_ENOMEM; }
+        group_off_cap_ = g.experts + 1;
+    }
+    cudaMemcpyAsync(group_off_host_, g.group_off, (size_t)(g.experts + 1) * sizeof(int), cudaMemcpyDeviceToHost, lane(k));
+    const int rc = b200_gather_rows(g.h, g.src_row, g.gathered, g.rows * g.top, D_, dtype_, lane(k));
+    if (rc != B200_OK) { err = "b200_gather_rows failed"; return rc; }
+    const cudaError_t e = cudaEventRecord(groups_ready_, lane(k));
+    if (e != cudaSuccess) { err = std::string("step: ") + cudaGetErrorString(e); return (int)e; }
+    return B200_OK;
+}
+
+int StepRunner::expert_products(const ExpertGroups& g, int k, std::string& err) {
+    const size_t ez = esz(), up_rows = (size_t)(g.epi == B200_GG_RELU2 || g.epi == B200_GG_NONE ? 1 : 2) * g.ff;
+    if (cudaEventSynchronize(groups_ready_) != cudaSuccess) { err = "step: the wait before the expert products failed"; return B200_EINVAL; }
+    for (cudaStream_t s : side_) cudaStreamWaitEvent(s, groups_ready_, 0);
+    int used = 0, rc = B200_OK;
+    for (int e = 0; e < g.experts; ++e) {
+        const int off = group_off_host_[e], n = group_off_host_[e + 1] - off;
+        if (n <= 0) continue;
+        cudaStream_t s = side_[used++ % kExpertStreams];
+        // no split-K workspace: the products of different streams run at the same time and must not share one
+        rc = b200_linear_ex((const char*)g.gathered + (size_t)off * D_ * ez, (const char*)g.w_up + (size_t)e * up_rows * D_ * ez,
+                            (char*)g.act + (size_t)off * g.ff * ez, n, g.ff, D_, dtype_, dtype_, g.epi, nullptr, 0, s);
+        if (rc == B200_OK)
+            rc = b200_linear_ex((const char*)g.act + (size_t)off * g.ff * ez, (const char*)g.w_down + (size_t)e * D_ * g.ff * ez,
+                                g.out + (size_t)off * D_, n, D_, g.ff, dtype_, B200_F32, B200_GG_NONE, nullptr, 0, s);
+        if (rc != B200_OK) { err = "expert product failed (" + std::to_string(rc) + ")"; break; }
+    }
+    for (int i = 0; i < kExpertStreams; ++i) {   // joined even after a failure: nothing of this step stays in flight behind the lane
+        cudaEventRecord(side_done_[i], side_[i]);
+        cudaStreamWaitEvent(lane(k), side_done_[i], 0);
+    }
+    return rc;
 }
 
 int StepRunner::step(const std::vector<StepEntry>& entries, float* logits_out, int* ids_out, std::string& err) {

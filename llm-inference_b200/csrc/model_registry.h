@@ -154,7 +154,33 @@ protected:
     size_t esz() const { return dtype_ == B200_BF16 ? 2 : 4; }
     void* dalloc(size_t bytes);   // device memory owned until the model closes
     // y[M, N] = A[M, K] W[N, K]^T, contiguous; A and W of the serving dtype: the tcgen05 GEMM when it fits, else the grouped one
-    int gemm(const void* A, const void* W, void* C, int c_dt, int M, int N, int K, int epi = B200_GG_NONE, float epi_param = 0.f);
+    int gemm(const void* A, const void* W, void* C, int c_dt, int M, int N, int K, int epi = B200_GG_NONE, float epi_param = 0.f,
+             int lane = 0);
+    // Lanes: lane 0 is stream_; sublayers that read the same input can run on lanes 1 .. kLanes - 1 beside it (captured into the
+    // step's graph as parallel branches). fork(lane) orders the lane behind everything on stream_, join(lane) the reverse. Every
+    // lane has its own split-K workspace.
+    static constexpr int kLanes = 3;
+    cudaStream_t lane(int k) const { return k == 0 ? stream_ : lanes_[k].stream; }
+    int fork(int k, std::string& err);
+    int join(int k, std::string& err);
+    // Routed experts of a prompt step. With hundreds of rows per expert the groups are dense GEMMs in their own right: the
+    // group sizes come to the host (one small copy and a wait: a prompt step is not captured into a graph), the sorted rows
+    // are gathered side by side, and every expert's up product (with its activation, `epi`; GLU epilogues: [gate; up] rows) and
+    // down product run on the tcgen05 GEMM, spread over side streams so that products of a few dozen tiles each fill the GPU
+    // together. Single-token steps and small prompts stay on the grouped kernel, which needs no host round trip.
+    // expert_rows() enqueues the copy and the gather on a lane; expert_products() waits for them on the host, enqueues the
+    // products and orders the lane behind them (other lanes can be given work in between).
+    struct ExpertGroups {
+        const void* h; int rows, top, experts, ff, epi;
+        const int* group_off; const int* src_row;
+        const void* w_up; const void* w_down;   // [experts, ff (GLU: 2 ff), D] and [experts, D, ff]
+        void* gathered; void* act; float* out;
+    };
+    bool experts_fit_streams(int rows, int ff, bool glu) const {
+        return dtype_ == B200_BF16 && !capturing_ && rows >= 1024 && D_ % 8 == 0 && ff % (glu ? 128 : 8) == 0;
+    }
+    int expert_rows(const ExpertGroups& g, int lane, std::string& err);
+    int expert_products(const ExpertGroups& g, int lane, std::string& err);
     // the host buffer of the logits follows the largest number of wanted places (called from ensure_scratch)
     int ensure_logits_host(int W);
     void buffers_moved() { ++buffers_epoch_; }   // a buffer that captured launches point into was reallocated
@@ -163,8 +189,6 @@ protected:
     int dtype_ = B200_BF16, vocab_ = 0, D_ = 0;
     SequenceBatch seq_;
     cudaStream_t stream_ = nullptr;
-    void* ws_ = nullptr;        // split-K partials of the weight-streaming GEMM
-    size_t ws_bytes_ = 0;
     void* attn_ws_ = nullptr;   // shares of split attention contexts / chunk summaries of a recurrence
     size_t attn_ws_bytes_ = 0;
     float* logits_ = nullptr;   // device, inside the family's scratch
@@ -173,6 +197,20 @@ protected:
 
 private:
     void drop_graphs();
+    struct Lane {
+        cudaStream_t stream = nullptr;              // lane 0 runs on stream_
+        cudaEvent_t forked = nullptr, joined = nullptr;
+        void* ws = nullptr;                         // split-K partials of the weight-streaming GEMM
+        size_t ws_bytes = 0;
+    };
+    Lane lanes_[kLanes];
+    // side streams of expert_products
+    static constexpr int kExpertStreams = 4;
+    std::vector<cudaStream_t> side_;
+    std::vector<cudaEvent_t> side_done_;
+    cudaEvent_t groups_ready_ = nullptr;
+    int* group_off_host_ = nullptr;   // pinned
+    int group_off_cap_ = 0;
     std::vector<void*> owned_;
     float* logits_host_ = nullptr;
     size_t logits_host_floats_ = 0;

@@ -1,5 +1,6 @@
 // Mixture-of-experts plumbing around b200_gemm_grouped: routers (softmax over all outputs with a corrected choice and
-// identity experts; or a choice on the biased logits with a softmax over the chosen ones), counting sort of the (token, choice) pairs by expert, and the fp32 residual update that gathers every
+// identity experts; a choice on the biased logits with a softmax over the chosen ones; or softmax over all with the choice
+// limited to the best groups of experts and renormalised weights), counting sort of the (token, choice) pairs by expert, and the fp32 residual update that gathers every
 // token's expert rows back in a fixed order (no atomics: a token's sum does not depend on the batch around it).
 #include "b200_serve.h"
 #include "common.cuh"
@@ -7,13 +8,79 @@
 
 namespace b200 {
 
+// index of the largest v[0..n) over a warp (ties: the lowest index); every lane gets it
+__device__ __forceinline__ int warp_argmax(const float* v, int n, int lane) {
+    float best = -INFINITY;
+    int at = n;
+    for (int i = lane; i < n; i += 32)
+        if (v[i] > best) { best = v[i]; at = i; }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+        const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+        const int oa = __shfl_xor_sync(0xffffffffu, at, o);
+        if (ob > best || (ob == best && oa < at)) { best = ob; at = oa; }
+    }
+    return min(at, n - 1);   // nothing above -inf (not-a-number logits): stays inside the table
+}
+
+// z[n_out] (logits, becomes the scores that may still be chosen), pick[n_out] scratch
+__device__ __forceinline__ void route_in_groups(float* z, float* pick, int n_out, int top, int groups, int keep, int lane, int* chosen,
+                                                float* weight) {
+    float m = -INFINITY, den = 0.f;
+    for (int o = lane; o < n_out; o += 32) m = fmaxf(m, z[o]);
+#pragma unroll
+    for (int s = 16; s > 0; s >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, s));
+    for (int o = lane; o < n_out; o += 32) {
+        z[o] = expf(z[o] - m);
+        den += z[o];
+    }
+#pragma unroll
+    for (int s = 16; s > 0; s >>= 1) den += __shfl_xor_sync(0xffffffffu, den, s);
+    const float inv = 1.0f / den;
+    for (int o = lane; o < n_out; o += 32) z[o] *= inv;
+    __syncwarp();
+    if (groups > 1) {
+        const int per = n_out / groups;
+        for (int q = lane; q < groups; q += 32) {
+            float b = -INFINITY;
+            for (int i = 0; i < per; ++i) b = fmaxf(b, z[q * per + i]);
+            pick[q] = b;
+        }
+        __syncwarp();
+        for (int k = 0; k < keep; ++k) {   // a kept group is marked with -inf: not found again, told apart below
+            const int q = warp_argmax(pick, groups, lane);
+            __syncwarp();
+            if (lane == 0) pick[q] = -INFINITY;
+            __syncwarp();
+        }
+        for (int o = lane; o < n_out; o += 32)
+            if (pick[o / per] != -INFINITY) z[o] = -1.f;   // scores are positive: never chosen before an allowed expert
+        __syncwarp();
+    }
+    float sum = 0.f;
+    for (int k = 0; k < top; ++k) {
+        const int e = warp_argmax(z, n_out, lane);
+        const float s = z[e];
+        __syncwarp();
+        if (lane == 0) {
+            z[e] = -2.f;
+            chosen[k] = e;
+            pick[k] = s;
+        }
+        sum += s;
+        __syncwarp();
+    }
+    for (int k = lane; k < top; k += 32) weight[k] = pick[k] / (sum + 1e-20f);
+}
+
 // one CTA per token: 16 warps compute the router outputs (fp32 dot over the width, eight loads in flight per lane),
 // thread 0 the softmax and the choice
 template <typename T>
 __global__ void __launch_bounds__(512) moe_route_kernel(const T* __restrict__ h, const float* __restrict__ wr,
                                                         const float* __restrict__ corr, const float* __restrict__ bias,
                                                         int on_logits, int width, int n_out, int top,
-                                                        float scale, int* __restrict__ chosen, float* __restrict__ weight) {
+                                                        float scale, int groups, int keep, int* __restrict__ chosen,
+                                                        float* __restrict__ weight) {
     extern __shared__ float z[];   // z[n_out] | pick[n_out] | x[width]
     float* pick = z + n_out;
     float* xs = pick + n_out;
@@ -47,6 +114,10 @@ __global__ void __launch_bounds__(512) moe_route_kernel(const T* __restrict__ h,
         if (lane == 0) z[o] = d + (bias ? bias[o] : 0.f);
     }
     __syncthreads();
+    if (groups > 0) {   // one warp: softmax, the best groups, the best experts inside them, renormalised weights
+        if (warp == 0) route_in_groups(z, pick, n_out, top, groups, keep, lane, chosen + (size_t)t * top, weight + (size_t)t * top);
+        return;
+    }
     if (threadIdx.x == 0 && on_logits) {   // the `top` largest logits, then a softmax over those alone
         float m = -INFINITY, den = 0.f;
         for (int k = 0; k < top; ++k) {
@@ -174,9 +245,9 @@ extern "C" int b200_moe_route(const void* h, int h_dtype, const float* w_router,
     if (smem > 48 * 1024) return B200_EUNSUPPORTED;
     if (h_dtype == B200_BF16)
         moe_route_kernel<__nv_bfloat16><<<n_tokens, 512, smem, s>>>((const __nv_bfloat16*)h, w_router, correction, nullptr, 0, width, n_out, top,
-                                                                   scale, chosen, weight);
+                                                                   scale, 0, 0, chosen, weight);
     else if (h_dtype == B200_F32)
-        moe_route_kernel<float><<<n_tokens, 512, smem, s>>>((const float*)h, w_router, correction, nullptr, 0, width, n_out, top, scale, chosen,
+        moe_route_kernel<float><<<n_tokens, 512, smem, s>>>((const float*)h, w_router, correction, nullptr, 0, width, n_out, top, scale, 0, 0, chosen,
                                                            weight);
     else
         return B200_EINVAL;
@@ -194,9 +265,31 @@ extern "C" int b200_moe_route_logits(const void* h, int h_dtype, const float* w_
     if (smem > 48 * 1024) return B200_EUNSUPPORTED;
     if (h_dtype == B200_BF16)
         moe_route_kernel<__nv_bfloat16><<<n_tokens, 512, smem, s>>>((const __nv_bfloat16*)h, w_router, nullptr, bias, 1, width, n_out, top, 1.f,
-                                                                   chosen, weight);
+                                                                   0, 0, chosen, weight);
     else if (h_dtype == B200_F32)
-        moe_route_kernel<float><<<n_tokens, 512, smem, s>>>((const float*)h, w_router, nullptr, bias, 1, width, n_out, top, 1.f, chosen, weight);
+        moe_route_kernel<float><<<n_tokens, 512, smem, s>>>((const float*)h, w_router, nullptr, bias, 1, width, n_out, top, 1.f, 0, 0, chosen, weight);
+    else
+        return B200_EINVAL;
+    count_launch();
+    return (int)cudaGetLastError();
+}
+
+extern "C" int b200_moe_route_groups(const void* h, int h_dtype, const float* w_router, int n_tokens, int width, int n_out, int top,
+                                     int groups, int keep, int* chosen, float* weight, void* stream) {
+    if (!h || !w_router || !chosen || !weight || n_tokens < 0 || width < 1 || n_out < 1 || top < 1 || groups < 1 || n_out % groups ||
+        keep < 1 || keep > groups || top > keep * (n_out / groups))
+        return B200_EINVAL;
+    if (n_out > 4096) return B200_EUNSUPPORTED;
+    if (n_tokens == 0) return B200_OK;
+    cudaStream_t s = (cudaStream_t)stream;
+    const size_t smem = ((size_t)2 * n_out + width) * sizeof(float);
+    if (smem > 48 * 1024) return B200_EUNSUPPORTED;
+    if (h_dtype == B200_BF16)
+        moe_route_kernel<__nv_bfloat16><<<n_tokens, 512, smem, s>>>((const __nv_bfloat16*)h, w_router, nullptr, nullptr, 0, width, n_out, top, 1.f,
+                                                                   groups, keep, chosen, weight);
+    else if (h_dtype == B200_F32)
+        moe_route_kernel<float><<<n_tokens, 512, smem, s>>>((const float*)h, w_router, nullptr, nullptr, 0, width, n_out, top, 1.f, groups, keep,
+                                                           chosen, weight);
     else
         return B200_EINVAL;
     count_launch();

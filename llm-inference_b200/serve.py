@@ -40,7 +40,7 @@ class PagedAttentionArgs(C.Structure):
                 ("scale", _f), ("softcap", _f), ("denom_bias", _f), ("dtype", _i), ("longest_entry", _i),
                 ("longest_context", _i), ("workspace", _vp), ("workspace_bytes", _sz),
                 ("chunk", _i), ("maps", _i), ("out_f32", _i),
-                ("window", _i), ("sigmoid_weights", _i), ("head_bias", _vp)]
+                ("window", _i), ("sigmoid_weights", _i), ("head_bias", _vp), ("head_temp", _vp), ("head_mix", _vp)]
 
 
 class RmsnormResidualArgs(C.Structure):
@@ -92,6 +92,28 @@ class GatedRecurrenceArgs(C.Structure):
                 ("workspace", _vp), ("workspace_bytes", _sz)]
 
 
+class LatentNormsArgs(C.Structure):
+    """mirror of ``b200_latent_norms_args``"""
+    _fields_ = [("raw", _vp), ("ld_raw", _ll), ("q_off", _i), ("kv_off", _i), ("q_norm", _vp), ("q_rank", _i), ("q_out", _vp),
+                ("kv_norm", _vp), ("eps", _f), ("pool", _vp), ("pages", _vp), ("max_pages", _i), ("page_rows", _i), ("slot", _vp), ("pos", _vp),
+                ("n_tokens", _i), ("rank", _i), ("extra", _i), ("cos", _vp), ("sin", _vp), ("rot_layout", _i), ("dtype", _i)]
+
+
+class ParallelResidualArgs(C.Structure):
+    """mirror of ``b200_parallel_residual_args``"""
+    _fields_ = [("x", _vp), ("mult", _f), ("y1", _vp), ("w1", _vp), ("s1", _f), ("y2", _vp), ("w2", _vp), ("s2", _f), ("y3", _vp),
+                ("expert_out", _vp), ("dest", _vp), ("weight", _vp), ("top", _i), ("ln_w", _vp), ("ln_b", _vp), ("eps", _f),
+                ("out", _vp), ("out_dtype", _i), ("n_rows", _i), ("width", _i)]
+
+
+class SsdScanArgs(C.Structure):
+    """mirror of ``b200_ssd_scan_args``"""
+    _fields_ = [("u", _vp), ("ld_u", _ll), ("x_off", _i), ("b_off", _i), ("c_off", _i), ("dt_raw", _vp), ("ld_dt", _ll), ("dt_bias", _vp),
+                ("A", _vp), ("D", _vp), ("state", _vp), ("out", _vp), ("ent_row", _vp), ("ent_len", _vp), ("slot", _vp), ("pos", _vp),
+                ("n_entries", _i), ("n_tokens", _i), ("heads", _i), ("groups", _i), ("vdim", _i), ("n_state", _i), ("longest_entry", _i),
+                ("chunked", _i), ("workspace", _vp), ("workspace_bytes", _sz)]
+
+
 class ModelOptions(C.Structure):
     """mirror of ``b200_model_options``"""
     _fields_ = [("dtype", _i), ("max_tokens", _i), ("max_slots", _i), ("max_step_tokens", _i)]
@@ -141,6 +163,14 @@ SERVE_PROTOTYPES = {
     "b200_embed_pair_hash": (_i, [_vp, _vp, _vp, _f, _vp, _i, _i, _i, _vp, _vp, _i, _i, _i, _vp]),
     "b200_scale": (_i, [_vp, _sz, _f, _vp]),
     "b200_glu_act_clamped": (_i, [_vp, _vp, _i, _i, _f, _i, _vp]),
+    "b200_moe_route_groups": (_i, [_vp, _i, _vp, _i, _i, _i, _i, _i, _i, _vp, _vp, _vp]),
+    "b200_parallel_residual": (_i, [C.POINTER(ParallelResidualArgs), _vp]),
+    "b200_poly_norm": (_i, [_vp, _vp, _f, _vp, _i, _i, _i, _vp]),
+    "b200_latent_norms": (_i, [C.POINTER(LatentNormsArgs), _vp]),
+    "b200_mixed_attention_workspace_bytes": (_sz, [_i, _i, _i, _i]),
+    "b200_ssd_scan_workspace_bytes": (_sz, [_i, _i, _i, _i, _i, _i]),
+    "b200_ssd_scan": (_i, [C.POINTER(SsdScanArgs), _vp]),
+    "b200_gated_group_rms": (_i, [_vp, _vp, _ll, _vp, _vp, _i, _i, _i, _f, _i, _vp]),
     "b200_serve_last_error": (C.c_char_p, []),
     "b200_model_families": (C.c_char_p, []),
     "b200_model_open": (_vp, [C.c_char_p, C.POINTER(ModelOptions)]),
