@@ -1,6 +1,6 @@
 """Prefill and decode throughput of a model family served through include/b200_serve.h, beside the LLaMA engine at
 equal size (same width, heads, layers, vocabulary and the same feed-forward width per token), random weights.
-Called by bench.py --workload nekodra | musilorn; prints one JSON line."""
+Called by bench.py --workload nekodra | musilorn | tomalix | sakevik | filipel; prints one JSON line."""
 import json
 import os
 import tempfile
@@ -63,6 +63,26 @@ SAKEVIK_SIZES = {
 }
 
 
+def filipel_layers(width, heads, kv_heads, dim, ff, expert_ff, window, q_rank, kv_rank, rot_dim, state, **_):
+    """four layers: latent attention with low-rank queries and a dense feed-forward; windowed attention mixed across heads
+    beside a state-space recurrence twice as wide as the model, with 16 experts of which a token uses 4 (two of four groups);
+    the same with a dense feed-forward; latent attention on the first layer's rows with routed experts"""
+    lat = dict(type="latent_attention", heads=heads, dim=dim, rot_dim=rot_dim, vdim=dim, q_rank=q_rank, kv_rank=kv_rank)
+    par = dict(type="parallel", left=dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=dim, window=window),
+               right=dict(heads=2 * width // 64, vdim=64, state=state, groups=1, conv=4, norm_groups=1))
+    moe = (expert_ff, 16, 4, 4, 2)
+    return [dict(lat, ff=ff), dict(par, ff=moe), dict(par, ff=ff), dict(lat, kv_from=0, ff=moe)]
+
+
+# expert_ff: a gated expert holds three matrices where a squared-relu expert of Tomalix holds two: two thirds of its width
+FILIPEL_SIZES = {
+    "s": dict(width=1024, heads=8, kv_heads=4, dim=128, ff=4096, expert_ff=640, window=1024, q_rank=512, kv_rank=256, rot_dim=64, state=128,
+              n_layers=4, vocab=32000),
+    "m": dict(width=2048, heads=16, kv_heads=8, dim=128, ff=8192, expert_ff=1408, window=1024, q_rank=1024, kv_rank=512, rot_dim=64, state=128,
+              n_layers=4, vocab=32000),
+}
+
+
 def timed(fn, steps, warmup):
     import torch
     for _ in range(warmup):
@@ -84,6 +104,8 @@ def run(pkg, size="m", prompt=2048, batch=8, context=1024, steps=10, warmup=3, d
         return run_tomalix(pkg, size, prompt, batch, context, steps, warmup, dtype)
     if family == "sakevik":
         return run_sakevik(pkg, size, prompt, batch, context, steps, warmup, dtype)
+    if family == "filipel":
+        return run_filipel(pkg, size, prompt, batch, context, steps, warmup, dtype)
     sz = (MUSILORN_SIZES if family == "musilorn" else SIZES)[size]
     rng = np.random.default_rng(0)
     out = {"workload": family, "size": size, "shape": sz, "prompt": prompt, "decode_batch": batch, "decode_context": context,
@@ -210,6 +232,29 @@ def run_sakevik(pkg, size, prompt, batch, context, steps, warmup, dtype):
            "dtype": dtype, "data": "synthetic ids, random weights", "timing": "host clock around synchronous steps (each step ends "
            "with the device-to-host copy of its results), after warm-up"}
     cfg, w = S.random_sakevik(sz["width"], sz["vocab"], sakevik_layers(**sz))
+    out.update(serve_family(S, cfg, w, prompt, batch, context, steps, warmup, dtype, sz["vocab"]))
+    del w
+    tx = dict(TOMALIX_SIZES[size])
+    try:
+        cfg, w = S.random_tomalix(tx["width"], tx["vocab"], tomalix_layers(**tx))
+        res = serve_family(S, cfg, w, prompt, batch, context, steps, warmup, dtype, tx["vocab"])
+        res["shape"] = tx
+        out["tomalix_equal_size"] = res
+    except Exception as ex:   # the comparison must not take the family's own numbers down
+        out["tomalix_equal_size"] = {"failed": f"{type(ex).__name__}: {ex}"}
+    return out
+
+
+def run_filipel(pkg, size, prompt, batch, context, steps, warmup, dtype):
+    """The Filipel family beside the closest existing one, Tomalix (the same serving layer and fp32 residual; a gated attention
+    with a mask beside a recurrence with carried state, dense and routed feed-forwards), at equal width, heads, head size,
+    layer count, vocabulary and feed-forward weights per layer."""
+    S = pkg.serve
+    sz = FILIPEL_SIZES[size]
+    out = {"workload": "filipel", "size": size, "shape": sz, "prompt": prompt, "decode_batch": batch, "decode_context": context,
+           "dtype": dtype, "data": "synthetic ids, random weights", "timing": "host clock around synchronous steps (each step ends "
+           "with the device-to-host copy of its results), after warm-up"}
+    cfg, w = S.random_filipel(sz["width"], sz["vocab"], filipel_layers(**sz))
     out.update(serve_family(S, cfg, w, prompt, batch, context, steps, warmup, dtype, sz["vocab"]))
     del w
     tx = dict(TOMALIX_SIZES[size])

@@ -3,7 +3,7 @@
 // over the keys that position i sees (causal, block mask, sliding window). Every head needs every other head's NORMALISED
 // weight of the same key, so nothing can run along the keys in one pass: the row's maxima and denominators come first.
 //
-//   mixed_attn_row_kernel   one CTA, or a cluster of up to eight CTAs that share the context, per token: ALL heads' scores of a
+//   mixed_attn_row_kernel   one CTA, or a cluster of up to sixteen CTAs that share the context, per token: ALL heads' scores of a
 //                           tile of keys in shared memory, the row statistics (exchanged through distributed shared memory
 //                           when several CTAs share the context), then weights, mix and weighted values, and the CTAs' partial
 //                           outputs added in rank order. A share of keys that fits one tile keeps its scores, a longer one
@@ -13,7 +13,7 @@
 //   to stay mostly in L2):
 //     mixed_scores_kernel   64 rows x one head per CTA: scores on mma.sync tiles -> fp32 workspace, row maxima and
 //                           denominators (online over the key tiles), and per row the range of columns it owns there;
-//     mixed_mix_kernel      a thread per (row, pair of keys): the heads' weights in registers, the mix in fp32, rounded to
+//     mixed_mix_kernel      a thread per (row, two or four keys): the heads' weights in registers, the mix in fp32, rounded to
 //                           bfloat16 only as the operand of the last product;
 //     mixed_values_kernel   64 rows x one head per CTA: weights times values on mma.sync tiles.
 #include <cooperative_groups.h>
@@ -30,12 +30,13 @@ namespace b200 {
 
 namespace cg = cooperative_groups;
 
-constexpr int kMxThreads = 256, kMxWarps = kMxThreads / 32, kMxMaxCluster = 8;
+constexpr int kMxThreads = 256, kMxWarps = kMxThreads / 32, kMxMaxCluster = 16;   // more than 8 CTAs per cluster: opt-in
 
 struct MxRow {
     PA a;
     int kt;        // keys per tile (a multiple of 4)
     int vec;       // rows of K can be read in 16-byte pieces
+    int vec4;      // rows of V can be read four values at a time
 };
 
 // scores of the tile's n keys (page rows in `rows`) for all heads; R heads of one key head share a pass over the key rows
@@ -108,6 +109,62 @@ __device__ __forceinline__ void mx_scores(const PA& a, const float* qs, const in
             for (int d = 0; d < dim; ++d) v = fmaf(q[d], DT<T>::to_f(kr[d]), v);
             sc[h * kt + kk] = v * pa_scale(a, h);
         }
+    }
+}
+
+template <typename T, int VC> struct MxVal;   // VC consecutive values of one key
+template <typename T> struct MxVal<T, 2> {
+    static __device__ __forceinline__ void load(const T* p, float (&v)[2]) {
+        const float2 t = Pair<T>::load(p);
+        v[0] = t.x; v[1] = t.y;
+    }
+};
+template <> struct MxVal<float, 4> {
+    static __device__ __forceinline__ void load(const float* p, float (&v)[4]) {
+        const float4 t = *reinterpret_cast<const float4*>(p);
+        v[0] = t.x; v[1] = t.y; v[2] = t.z; v[3] = t.w;
+    }
+};
+template <> struct MxVal<__nv_bfloat16, 4> {
+    static __device__ __forceinline__ void load(const __nv_bfloat16* p, float (&v)[4]) {
+        const uint2 t = *reinterpret_cast<const uint2*>(p);
+        const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&t.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&t.y));
+        v[0] = a.x; v[1] = a.y; v[2] = b.x; v[3] = b.y;
+    }
+};
+// om += mixed weights times values over the tile's n keys: a thread per VC value columns and R heads of one key head
+template <typename T, int R, int VC>
+__device__ __forceinline__ void mx_values(const T* V, const int* rows, const float* mx, float* om, int H, int G, int dv, int kt, int n) {
+    const int hv = dv / VC, per = H / G;
+    for (int i = threadIdx.x; i < (H / R) * hv; i += kMxThreads) {
+        const int u = i / hv, c = VC * (i - u * hv), g = u * R / per;
+        const float* w = mx + u * R * kt;
+        float acc[R][VC];
+#pragma unroll
+        for (int r = 0; r < R; ++r)
+#pragma unroll
+            for (int x = 0; x < VC; ++x) acc[r][x] = 0.f;
+        constexpr int F = R <= 4 ? 8 : 4;   // keys whose values are in flight together
+        for (int k = 0; k < n; k += F) {
+            float v[F][VC];
+#pragma unroll
+            for (int y = 0; y < F; ++y) MxVal<T, VC>::load(V + ((size_t)rows[min(k + y, n - 1)] * G + g) * dv + c, v[y]);
+#pragma unroll
+            for (int y0 = 0; y0 < F; y0 += 4) {
+                if (k + y0 >= n) break;
+#pragma unroll
+                for (int r = 0; r < R; ++r) {
+                    const float4 w4 = *reinterpret_cast<const float4*>(w + r * kt + k + y0);
+#pragma unroll
+                    for (int x = 0; x < VC; ++x)
+                        acc[r][x] = fmaf(w4.w, v[y0 + 3][x], fmaf(w4.z, v[y0 + 2][x], fmaf(w4.y, v[y0 + 1][x], fmaf(w4.x, v[y0][x], acc[r][x]))));
+                }
+            }
+        }
+#pragma unroll
+        for (int r = 0; r < R; ++r)
+#pragma unroll
+            for (int x = 0; x < VC; ++x) om[(u * R + r) * dv + c + x] += acc[r][x];
     }
 }
 
@@ -197,31 +254,10 @@ __global__ void __launch_bounds__(kMxThreads) mixed_attn_row_kernel(const MxRow 
             mx[h * kt + k] = v;   // places behind the last key are 0
         }
         __syncthreads();
-        if ((dv & 1) == 0) {      // a thread per pair of value columns and R heads
-            const int hv = dv / 2;
-            for (int i = threadIdx.x; i < (H / R) * hv; i += kMxThreads) {
-                const int u = i / hv, c = 2 * (i - u * hv), g = u * R / per;
-                const float* w = mx + u * R * kt;
-                float acc[R][2];
-#pragma unroll
-                for (int r = 0; r < R; ++r) acc[r][0] = acc[r][1] = 0.f;
-#pragma unroll 2
-                for (int k = 0; k < n; k += 4) {
-                    float2 v[4];
-#pragma unroll
-                    for (int x = 0; x < 4; ++x) v[x] = Pair<T>::load(V + ((size_t)rows[min(k + x, n - 1)] * G + g) * dv + c);
-#pragma unroll
-                    for (int r = 0; r < R; ++r) {
-                        const float4 w4 = *reinterpret_cast<const float4*>(w + r * kt + k);
-                        acc[r][0] = fmaf(w4.x, v[0].x, acc[r][0]); acc[r][1] = fmaf(w4.x, v[0].y, acc[r][1]);
-                        acc[r][0] = fmaf(w4.y, v[1].x, acc[r][0]); acc[r][1] = fmaf(w4.y, v[1].y, acc[r][1]);
-                        acc[r][0] = fmaf(w4.z, v[2].x, acc[r][0]); acc[r][1] = fmaf(w4.z, v[2].y, acc[r][1]);
-                        acc[r][0] = fmaf(w4.w, v[3].x, acc[r][0]); acc[r][1] = fmaf(w4.w, v[3].y, acc[r][1]);
-                    }
-                }
-#pragma unroll
-                for (int r = 0; r < R; ++r) { om[(u * R + r) * dv + c] += acc[r][0]; om[(u * R + r) * dv + c + 1] += acc[r][1]; }
-            }
+        if (dv % 4 == 0 && m.vec4)
+            mx_values<T, R, 4>(V, rows, mx, om, H, G, dv, kt, n);
+        else if (dv % 2 == 0) {
+            mx_values<T, R, 2>(V, rows, mx, om, H, G, dv, kt, n);
         } else {
             for (int i = threadIdx.x; i < H * dv; i += kMxThreads) {
                 const int h = i / dv, c = i - h * dv, g = h / per;
@@ -253,6 +289,14 @@ template <typename T, int R>
 static int launch_mx_row(MxRow m, int cluster, size_t smem, cudaStream_t s) {
     static unsigned long long done = 0;
     cudaError_t e = ensure_max_dynamic_smem((const void*)mixed_attn_row_kernel<T, R>, (int)kMxSmem, done);
+    if (e == cudaSuccess && cluster > 8) {
+        static unsigned long long wide = 0;
+        const int dev = current_device();
+        if (!(wide & (1ull << dev))) {
+            e = cudaFuncSetAttribute((const void*)mixed_attn_row_kernel<T, R>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
+            if (e == cudaSuccess) wide |= 1ull << dev;
+        }
+    }
     if (e != cudaSuccess) return (int)e;
     cudaLaunchConfig_t cfg{};
     cfg.gridDim = dim3((unsigned)m.a.n_tokens * cluster);
@@ -338,6 +382,9 @@ __global__ void __launch_bounds__(128) mixed_scores_kernel(const MxTile m) {
     const bf* Kp = reinterpret_cast<const bf*>(a.k_pool);
     const int r_lo = warp * 16 + gid, r_hi = r_lo + 8;
     const float sc_h = pa_scale(a, h);
+    // a thread keeps its 16-byte column of a key tile when the columns divide the threads and a page holds whole tiles
+    const bool one_page = a.page_rows % kMxTile == 0 && 128 % CH == 0;
+    const int c_own = (threadIdx.x % CH) * 8, r_own = threadIdx.x / CH, r_step = 128 / CH;
     float m_run[2] = {-1e30f, -1e30f}, l_run[2] = {0.f, 0.f};
     for (int seg = 0; seg < rows;) {
         const MxSeg sg = mx_segment(a, row_pos, row_slot, rows, seg);
@@ -351,12 +398,20 @@ __global__ void __launch_bounds__(128) mixed_scores_kernel(const MxTile m) {
                 m.range[l0 + r] = make_int2(sg.base, (sg.n_keys - sg.base + kMxTile - 1) / kMxTile * kMxTile);
         auto load_tile = [&](int k0, int buf) {
             bf* kd = Ks + buf * kMxTile * RS;
-            for (int i = threadIdx.x; i < kMxTile * CH; i += blockDim.x) {
-                const int kr = i / CH, c = (i - kr * CH) * 8, j = k0 + kr;
-                const bool ok = j < sg.n_keys && c < dim;
-                const size_t row = ok ? (size_t)plist[j / a.page_rows] * a.page_rows + j % a.page_rows : 0;
-                mx_cp16(kd + kr * RS + c, Kp + (row * G + g) * dim + (ok ? c : 0), ok);
-            }
+            if (one_page) {   // whole rows per step of the threads: one lookup, no divisions
+                const size_t row = (size_t)plist[k0 / a.page_rows] * a.page_rows + k0 % a.page_rows;
+                const bf* src = Kp + (row * G + g) * dim + c_own;
+                for (int kr = r_own; kr < kMxTile; kr += r_step) {
+                    const bool ok = k0 + kr < sg.n_keys && c_own < dim;
+                    mx_cp16(kd + kr * RS + c_own, ok ? src + (size_t)kr * G * dim : Kp, ok);
+                }
+            } else
+                for (int i = threadIdx.x; i < kMxTile * CH; i += blockDim.x) {
+                    const int kr = i / CH, c = (i - kr * CH) * 8, j = k0 + kr;
+                    const bool ok = j < sg.n_keys && c < dim;
+                    const size_t row = ok ? (size_t)plist[j / a.page_rows] * a.page_rows + j % a.page_rows : 0;
+                    mx_cp16(kd + kr * RS + c, Kp + (row * G + g) * dim + (ok ? c : 0), ok);
+                }
             asm volatile("cp.async.commit_group;" ::: "memory");
         };
         __syncthreads();   // the buffers of the previous segment are no longer read
@@ -423,51 +478,77 @@ __global__ void __launch_bounds__(128) mixed_scores_kernel(const MxTile m) {
     }
 }
 
-template <int HP>   // heads rounded up: 8, 16, 32 or 64 (a multiple of 4)
+template <int CW> struct MxCols;   // CW consecutive columns of one head
+template <> struct MxCols<2> {
+    static __device__ __forceinline__ void load(const float* p, float (&v)[2]) {
+        const float2 t = *reinterpret_cast<const float2*>(p);
+        v[0] = t.x; v[1] = t.y;
+    }
+    static __device__ __forceinline__ void store(__nv_bfloat16* p, const float (&v)[2]) {
+        *reinterpret_cast<uint32_t*>(p) = pa_pack(v[0], v[1]);
+    }
+};
+template <> struct MxCols<4> {
+    static __device__ __forceinline__ void load(const float* p, float (&v)[4]) {
+        const float4 t = *reinterpret_cast<const float4*>(p);
+        v[0] = t.x; v[1] = t.y; v[2] = t.z; v[3] = t.w;
+    }
+    static __device__ __forceinline__ void store(__nv_bfloat16* p, const float (&v)[4]) {
+        *reinterpret_cast<uint2*>(p) = make_uint2(pa_pack(v[0], v[1]), pa_pack(v[2], v[3]));
+    }
+};
+
+template <int HP, int CW>   // heads rounded up (8, 16, 32 or 64), columns per thread
 __global__ void __launch_bounds__(128) mixed_mix_kernel(const MxTile m) {
     extern __shared__ __align__(16) float tk[];   // [heads][HP] mix, columns behind the last head zero; then [heads] (max, 1 / den)
     const PA& a = m.a;
     const int H = a.heads, l = blockIdx.x;
     const int2 rg = m.range[l];
-    if (blockIdx.y * 256 >= rg.y) return;
+    if (blockIdx.y * 128 * CW >= rg.y) return;
     float2* st = reinterpret_cast<float2*>(tk + H * HP);
     for (int i = threadIdx.x; i < H * HP; i += 128) {
         const int h = i / HP, g = i % HP;
         tk[i] = g < H ? a.head_mix[h * H + g] : 0.f;
     }
     for (int i = threadIdx.x; i < H; i += 128) st[i] = m.stat[(size_t)l * H + i];
-    __syncthreads();
-    const int col = blockIdx.y * 256 + 2 * threadIdx.x;
-    if (col >= rg.y) return;
+    const int col = (blockIdx.y * 128 + threadIdx.x) * CW;
+    const bool mine = col < rg.y;                 // whole tiles of 64 columns: a thread's columns are all inside or all outside
     const int p = a.pos[m.row0 + l], f = pa_first_key(a, p), j = rg.x + col;
-    const bool in0 = j >= f && j <= p, in1 = j + 1 >= f && j + 1 <= p;
+    const bool any = mine && j + CW > f && j <= p;
     const size_t row = (size_t)l * H * m.width + col;
-    __nv_bfloat16* dst = m.w + row;
-    if (!in0 && !in1) {   // the tile reaches beyond what the row sees: weights of zero
-        for (int h = 0; h < H; ++h) *reinterpret_cast<__nv_bfloat162*>(dst + (size_t)h * m.width) = __floats2bfloat162_rn(0.f, 0.f);
-        return;
-    }
-    float w0[HP], w1[HP];
+    float w[HP][CW];
 #pragma unroll
     for (int g = 0; g < HP; ++g) {
-        w0[g] = w1[g] = 0.f;
-        if (g < H) {
-            const float2 s = *reinterpret_cast<const float2*>(m.s + row + (size_t)g * m.width);
-            w0[g] = in0 ? __expf(s.x - st[g].x) * st[g].y : 0.f;
-            w1[g] = in1 ? __expf(s.y - st[g].x) * st[g].y : 0.f;
-        }
+#pragma unroll
+        for (int c = 0; c < CW; ++c) w[g][c] = 0.f;
+        if (any && g < H) MxCols<CW>::load(m.s + row + (size_t)g * m.width, w[g]);
+    }
+    __syncthreads();
+    if (!mine) return;
+    __nv_bfloat16* dst = m.w + row;
+    if (any) {
+#pragma unroll
+        for (int g = 0; g < HP; ++g)
+            if (g < H) {
+                const float2 sg = st[g];
+#pragma unroll
+                for (int c = 0; c < CW; ++c) w[g][c] = (j + c >= f && j + c <= p) ? __expf(w[g][c] - sg.x) * sg.y : 0.f;
+            }
     }
     for (int h = 0; h < H; ++h) {
-        float v0 = 0.f, v1 = 0.f;
+        float v[CW];
 #pragma unroll
-        for (int g = 0; g < HP; g += 4) {
-            const float4 k4 = *reinterpret_cast<const float4*>(tk + h * HP + g);
-            v0 = fmaf(k4.x, w0[g], v0); v1 = fmaf(k4.x, w1[g], v1);
-            v0 = fmaf(k4.y, w0[g + 1], v0); v1 = fmaf(k4.y, w1[g + 1], v1);
-            v0 = fmaf(k4.z, w0[g + 2], v0); v1 = fmaf(k4.z, w1[g + 2], v1);
-            v0 = fmaf(k4.w, w0[g + 3], v0); v1 = fmaf(k4.w, w1[g + 3], v1);
+        for (int c = 0; c < CW; ++c) v[c] = 0.f;
+        if (any) {
+#pragma unroll
+            for (int g = 0; g < HP; g += 4) {
+                const float4 k4 = *reinterpret_cast<const float4*>(tk + h * HP + g);
+#pragma unroll
+                for (int c = 0; c < CW; ++c)
+                    v[c] = fmaf(k4.w, w[g + 3][c], fmaf(k4.z, w[g + 2][c], fmaf(k4.y, w[g + 1][c], fmaf(k4.x, w[g][c], v[c]))));
+            }
         }
-        *reinterpret_cast<__nv_bfloat162*>(dst + (size_t)h * m.width) = __floats2bfloat162_rn(v0, v1);
+        MxCols<CW>::store(dst + (size_t)h * m.width, v);   // columns that the row does not see: weights of zero
     }
 }
 
@@ -506,10 +587,13 @@ __global__ void __launch_bounds__(128) mixed_values_kernel(const MxTile m) {
                 const bool ok = r >= seg && r < sg.end;   // rows of other sequences: zero weights
                 mx_cp16(wd + r * PS + c, m.w + ((size_t)(l0 + (ok ? r : 0)) * a.heads + h) * m.width + (ok ? k0 - sg.base + c : 0), ok);
             }
-            for (int i = threadIdx.x; i < kMxTile * NT; i += blockDim.x) {
+            const bool one_page = a.page_rows % kMxTile == 0;
+            const size_t base = one_page ? (size_t)plist[k0 / a.page_rows] * a.page_rows + k0 % a.page_rows : 0;
+#pragma unroll
+            for (int i = threadIdx.x; i < kMxTile * NT; i += 128) {
                 const int kr = i / NT, c = (i - kr * NT) * 8, j = k0 + kr;
                 const bool ok = j < sg.n_keys && c < dv;
-                const size_t row = ok ? (size_t)plist[j / a.page_rows] * a.page_rows + j % a.page_rows : 0;
+                const size_t row = !ok ? 0 : one_page ? base + kr : (size_t)plist[j / a.page_rows] * a.page_rows + j % a.page_rows;
                 mx_cp16(vd + kr * RSV + c, Vp + (row * G + g) * dv + (ok ? c : 0), ok);
             }
             asm volatile("cp.async.commit_group;" ::: "memory");
@@ -560,7 +644,7 @@ static long long mx_width(int span, int longest) {
     return span > 0 ? std::min(all, ((long long)span + 2 * kMxTile - 2 + kMxTile - 1) / kMxTile * kMxTile) : all;
 }
 static size_t mx_row_bytes(int heads, long long width) { return (size_t)heads * width * 6 + (size_t)heads * 8 + 8; }
-constexpr size_t kMxBlockBytes = 128ull << 20, kMxMostBytes = 1024ull << 20;   // a block of rows: mostly L2; never more than 1 GB
+constexpr size_t kMxBlockBytes = 256ull << 20, kMxMostBytes = 1024ull << 20;   // a block of rows: mostly L2; never more than 1 GB
 
 // rows per block: whole tiles
 static int mx_block_rows(int n_tokens, size_t row_bytes) {
@@ -597,12 +681,12 @@ static int mixed_tiles(const PA& a, int span, int longest_context, void* workspa
         m.n_rows = std::min(block, a.n_tokens - m.row0);
         const dim3 grid((m.n_rows + kMxTile - 1) / kMxTile, a.heads);
         mixed_scores_kernel<<<grid, 128, sm1, s>>>(m);
-        const dim3 gm(m.n_rows, (unsigned)((width + 255) / 256));
+        const dim3 gm4(m.n_rows, (unsigned)((width + 511) / 512)), gm2(m.n_rows, (unsigned)((width + 255) / 256));
         auto mix_smem = [&](int hp) { return (size_t)a.heads * hp * 4 + (size_t)a.heads * 8; };
-        if (a.heads <= 8) mixed_mix_kernel<8><<<gm, 128, mix_smem(8), s>>>(m);
-        else if (a.heads <= 16) mixed_mix_kernel<16><<<gm, 128, mix_smem(16), s>>>(m);
-        else if (a.heads <= 32) mixed_mix_kernel<32><<<gm, 128, mix_smem(32), s>>>(m);
-        else mixed_mix_kernel<64><<<gm, 128, mix_smem(64), s>>>(m);
+        if (a.heads <= 8) mixed_mix_kernel<8, 4><<<gm4, 128, mix_smem(8), s>>>(m);
+        else if (a.heads <= 16) mixed_mix_kernel<16, 4><<<gm4, 128, mix_smem(16), s>>>(m);
+        else if (a.heads <= 32) mixed_mix_kernel<32, 4><<<gm4, 128, mix_smem(32), s>>>(m);
+        else mixed_mix_kernel<64, 2><<<gm2, 128, mix_smem(64), s>>>(m);
         const int rc = a.vdim <= 32 ? launch_values<4>(m, grid, s) : a.vdim <= 64 ? launch_values<8>(m, grid, s)
                        : a.vdim <= 128 ? launch_values<16>(m, grid, s) : launch_values<32>(m, grid, s);
         if (rc != 0) return rc;
@@ -632,7 +716,7 @@ int mixed_attention(const PA& a, int dtype, int longest_entry, int longest_conte
     if (fixed + 8 * per_key > kMxSmem) return B200_EUNSUPPORTED;
     const int share = ((seen + cluster - 1) / cluster + 3) & ~3;
     const int kt = (int)std::min<size_t>(std::min(share, 512), (kMxSmem - fixed) / per_key) & ~3;
-    MxRow m{a, kt, a.dim % 8 == 0 && al16(a.k_pool)};
+    MxRow m{a, kt, a.dim % 8 == 0 && al16(a.k_pool), al16(a.v_pool)};
     const size_t smem = fixed + (size_t)kt * per_key;
     return dtype == B200_BF16 ? launch_mx_row_for<__nv_bfloat16>(m, cluster, smem, s) : launch_mx_row_for<float>(m, cluster, smem, s);
 }

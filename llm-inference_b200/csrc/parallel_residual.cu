@@ -42,7 +42,7 @@ __global__ void __launch_bounds__(THREADS) parallel_residual_reg_kernel(const b2
         }
         __syncthreads();
     }
-    float v[kPrPer], p1[kPrPer], p2[kPrPer], p3[kPrPer], lw[kPrPer], lb[kPrPer];
+    float v[kPrPer], p1[kPrPer], p2[kPrPer], p3[kPrPer], w1[kPrPer], w2[kPrPer], lw[kPrPer], lb[kPrPer];
 #pragma unroll
     for (int k = 0; k < kPrPer; ++k) {
         const int c = threadIdx.x + THREADS * k;
@@ -51,18 +51,22 @@ __global__ void __launch_bounds__(THREADS) parallel_residual_reg_kernel(const b2
         p1[k] = (in && a.y1) ? a.y1[base + c] : 0.f;
         p2[k] = (in && a.y2) ? a.y2[base + c] : 0.f;
         p3[k] = (in && a.y3) ? a.y3[base + c] : 0.f;
+        w1[k] = (in && a.w1) ? a.w1[c] : 1.f;
+        w2[k] = (in && a.w2) ? a.w2[c] : 1.f;
         lw[k] = (in && a.ln_w) ? a.ln_w[c] : 0.f;
         lb[k] = (in && a.ln_b) ? a.ln_b[c] : 0.f;
     }
     if (a.expert_out) {
+#pragma unroll 2
+        for (int j = 0; j < a.top; ++j) {   // an expert's row at a time: its loads are in flight together
+            const int d = e_dest[j];
+            if (d < 0) continue;
+            const float* er = a.expert_out + (size_t)d * width;
+            float e[kPrPer];
 #pragma unroll
-        for (int k = 0; k < kPrPer; ++k) {
-            const int c = threadIdx.x + THREADS * k;
-            float r = 0.f;
-            if (c < width)
-                for (int j = 0; j < a.top; ++j)
-                    if (e_dest[j] >= 0) r = fmaf(e_w[j], a.expert_out[(size_t)e_dest[j] * width + c], r);
-            p3[k] += r;
+            for (int k = 0; k < kPrPer; ++k) e[k] = threadIdx.x + THREADS * k < width ? er[threadIdx.x + THREADS * k] : 0.f;
+#pragma unroll
+            for (int k = 0; k < kPrPer; ++k) p3[k] = fmaf(e_w[j], e[k], p3[k]);
         }
     }
     float r1 = 1.f, r2 = 1.f;
@@ -80,8 +84,8 @@ __global__ void __launch_bounds__(THREADS) parallel_residual_reg_kernel(const b2
         const int c = threadIdx.x + THREADS * k;
         if (c < width) {
             float y = 0.f;
-            if (a.y1) y += a.s1 * (a.w1 ? p1[k] * r1 * a.w1[c] : p1[k]);
-            if (a.y2) y += a.s2 * (a.w2 ? p2[k] * r2 * a.w2[c] : p2[k]);
+            if (a.y1) y += a.s1 * (p1[k] * r1 * w1[k]);   // no norm: both factors are 1
+            if (a.y2) y += a.s2 * (p2[k] * r2 * w2[k]);
             y += p3[k];
             v[k] += a.mult * y;
             a.x[base + c] = v[k];
@@ -127,14 +131,11 @@ __global__ void __launch_bounds__(256) parallel_residual_kernel(const b200_paral
     float sum = 0.f;
     for (int c = threadIdx.x; c < width; c += 256) {
         float y = 0.f, r = a.y3 ? a.y3[base + c] : 0.f;
-        if (a.expert_out) {
-            float e = 0.f;
+        if (a.expert_out)
             for (int j = 0; j < a.top; ++j) {
                 const int d = a.dest[(size_t)i * a.top + j];
-                if (d >= 0) e = fmaf(a.weight[(size_t)i * a.top + j], a.expert_out[(size_t)d * width + c], e);
+                if (d >= 0) r = fmaf(a.weight[(size_t)i * a.top + j], a.expert_out[(size_t)d * width + c], r);
             }
-            r += e;
-        }
         if (a.y1) y += a.s1 * (a.w1 ? a.y1[base + c] * r1 * a.w1[c] : a.y1[base + c]);
         if (a.y2) y += a.s2 * (a.w2 ? a.y2[base + c] * r2 * a.w2[c] : a.y2[base + c]);
         y += r;

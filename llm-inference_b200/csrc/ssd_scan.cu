@@ -151,23 +151,28 @@ __device__ __forceinline__ void ssd_chunk_sums(const SS& a, int h, int row0, int
     }
 }
 
-// `rows` rows of `cols` columns from global (leading dimension ld) into shared memory rounded to tf32, rows beyond `live` and
-// columns beyond cols (up to cpad) zero
+// `rows` rows of `cols` columns from global (leading dimension ld) into shared memory, rows beyond `live` and columns beyond
+// cols (up to cpad) zero. Rows that allow it travel by cp.async (nothing waits for a load here: ssd_landed() before the first
+// read); the values are rounded to tf32 when a fragment picks them up.
 __device__ __forceinline__ void ssd_stage(float* dst, int stride, const float* src, long long ld, int rows, int live, int cols, int cpad) {
     if ((cols & 3) == 0 && (ld & 3) == 0 && (reinterpret_cast<uintptr_t>(src) & 15u) == 0 && cpad == cols) {
         const int q = cols / 4;
         for (int i = threadIdx.x; i < rows * q; i += blockDim.x) {
             const int r = i / q, c = (i - r * q) * 4;
-            float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (r < live) v = *reinterpret_cast<const float4*>(src + (size_t)r * ld + c);
-            *reinterpret_cast<float4*>(dst + r * stride + c) = make_float4(ssd_tf32(v.x), ssd_tf32(v.y), ssd_tf32(v.z), ssd_tf32(v.w));
+            const uint32_t d = (uint32_t)__cvta_generic_to_shared(dst + r * stride + c);
+            const float* g = src + (r < live ? (size_t)r * ld + c : 0);
+            asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(d), "l"(g), "r"(r < live ? 16 : 0) : "memory");
         }
         return;
     }
     for (int i = threadIdx.x; i < rows * cpad; i += blockDim.x) {
         const int r = i / cpad, c = i - r * cpad;
-        dst[r * stride + c] = (r < live && c < cols) ? ssd_tf32(src[(size_t)r * ld + c]) : 0.f;
+        dst[r * stride + c] = (r < live && c < cols) ? src[(size_t)r * ld + c] : 0.f;
     }
+}
+__device__ __forceinline__ void ssd_landed() {
+    asm volatile("cp.async.commit_group;\n\tcp.async.wait_group 0;" ::: "memory");
+    __syncthreads();
 }
 
 struct SsdChunk {
@@ -189,18 +194,18 @@ __global__ void __launch_bounds__(128) ssd_cb_kernel(const SS a) {
     const float* row = a.u + (size_t)ck.row0 * a.ld_u + g * N;
     ssd_stage(Cs, st, row + a.c_off, a.ld_u, kSsdChunk, ck.len, N, npad);
     ssd_stage(Bs, st, row + a.b_off, a.ld_u, kSsdChunk, ck.len, N, npad);
-    __syncthreads();
+    ssd_landed();
     const int warp = threadIdx.x / 32, lane = threadIdx.x % 32, gid = lane >> 2, tig = lane & 3, m0 = warp * 16;
     float acc[8][4];
 #pragma unroll
     for (int nt = 0; nt < 8; ++nt) acc[nt][0] = acc[nt][1] = acc[nt][2] = acc[nt][3] = 0.f;
     for (int k0 = 0; k0 < npad; k0 += 8) {
         const float* ar = Cs + (m0 + gid) * st + k0 + tig;
-        const float av[4] = {ar[0], ar[8 * st], ar[4], ar[8 * st + 4]};
+        const float av[4] = {ssd_tf32(ar[0]), ssd_tf32(ar[8 * st]), ssd_tf32(ar[4]), ssd_tf32(ar[8 * st + 4])};
 #pragma unroll
         for (int nt = 0; nt < 8; ++nt) {
             const float* br = Bs + (nt * 8 + gid) * st + k0 + tig;
-            ssd_mma(acc[nt], av, br[0], br[4]);
+            ssd_mma(acc[nt], av, ssd_tf32(br[0]), ssd_tf32(br[4]));
         }
     }
     float* dst = a.chunk_cb + ((size_t)ck.place * a.groups + g) * kSsdChunk * kSsdChunk;
@@ -220,18 +225,23 @@ __global__ void __launch_bounds__(128) ssd_state_kernel(const SS a) {
     const SsdChunk ck = ssd_chunk_of(a, e, blockIdx.y);
     if (!ck.on) return;
     const int h = blockIdx.z, g = h / (a.heads / a.groups), N = a.n_state, P = a.vdim, npad = (N + 15) & ~15, st = ssd_stride8(npad);
-    float* Xs = sm;                        // [64][kSsdXs]: dt_j exp(cum_end - cum_j) x_j
+    float* Xs = sm;                        // [64][kSsdXs]
     float* Bs = sm + kSsdChunk * kSsdXs;   // [64][st]
+    const int cols = min(kSsdCols, P - p0);
+    const float* row = a.u + (size_t)ck.row0 * a.ld_u;
+    ssd_stage(Bs, st, row + a.b_off + g * N, a.ld_u, kSsdChunk, ck.len, N, npad);
+    ssd_stage(Xs, kSsdXs, row + a.x_off + h * P + p0, a.ld_u, kSsdChunk, ck.len, cols, kSsdCols);
     ssd_chunk_sums(a, h, ck.row0, ck.len, dts, cum);
-    ssd_stage(Bs, st, a.u + (size_t)ck.row0 * a.ld_u + a.b_off + g * N, a.ld_u, kSsdChunk, ck.len, N, npad);
-    __syncthreads();
+    ssd_landed();
     if (threadIdx.x < kSsdChunk) wts[threadIdx.x] = dts[threadIdx.x] * expf((float)(cum[kSsdChunk - 1] - cum[threadIdx.x]));
     if (threadIdx.x == 0 && p0 == 0) a.chunk_decay[(size_t)ck.place * a.heads + h] = expf((float)cum[kSsdChunk - 1]);
     __syncthreads();
-    const float* xr = a.u + (size_t)ck.row0 * a.ld_u + a.x_off + h * P + p0;
-    for (int i = threadIdx.x; i < kSsdChunk * kSsdCols; i += 128) {
-        const int j = i / kSsdCols, p = i % kSsdCols;
-        Xs[j * kSsdXs + p] = (j < ck.len && p0 + p < P) ? ssd_tf32(xr[(size_t)j * a.ld_u + p] * wts[j]) : 0.f;
+    // the weights dt_j exp(cum_end - cum_j) go into the value rows, in place
+    for (int i = threadIdx.x; i < kSsdChunk * (kSsdCols / 4); i += 128) {
+        float4* x4 = reinterpret_cast<float4*>(Xs + (i / (kSsdCols / 4)) * kSsdXs) + i % (kSsdCols / 4);
+        const float w = wts[i / (kSsdCols / 4)];
+        const float4 v = *x4;
+        *x4 = make_float4(ssd_tf32(v.x * w), ssd_tf32(v.y * w), ssd_tf32(v.z * w), ssd_tf32(v.w * w));
     }
     __syncthreads();
     const int warp = threadIdx.x / 32, lane = threadIdx.x % 32, gid = lane >> 2, tig = lane & 3;
@@ -241,10 +251,10 @@ __global__ void __launch_bounds__(128) ssd_state_kernel(const SS a) {
         float acc[8][4];
 #pragma unroll
         for (int nt = 0; nt < 8; ++nt) acc[nt][0] = acc[nt][1] = acc[nt][2] = acc[nt][3] = 0.f;
-#pragma unroll
+#pragma unroll 2
         for (int k0 = 0; k0 < kSsdChunk; k0 += 8) {
             const float* ar = Bs + (k0 + tig) * st + m0 + gid;
-            const float av[4] = {ar[0], ar[8], ar[4 * st], ar[4 * st + 8]};
+            const float av[4] = {ssd_tf32(ar[0]), ssd_tf32(ar[8]), ssd_tf32(ar[4 * st]), ssd_tf32(ar[4 * st + 8])};
             const float* br = Xs + (k0 + tig) * kSsdXs + gid;
 #pragma unroll
             for (int nt = 0; nt < 8; ++nt) ssd_mma(acc[nt], av, br[nt * 8], br[4 * kSsdXs + nt * 8]);
@@ -265,28 +275,43 @@ __global__ void __launch_bounds__(128) ssd_state_kernel(const SS a) {
     }
 }
 
-// element-wise over the state: walks the entry's chunks, leaves S at each chunk's start in place of its U
-__global__ void __launch_bounds__(256) ssd_carry_kernel(const SS a) {
-    const int e = blockIdx.x, h = blockIdx.y, i = blockIdx.z * blockDim.x + threadIdx.x, per = a.n_state * a.vdim;
+// element-wise over the state (VEC consecutive elements per thread): walks the entry's chunks, leaves S at each chunk's start in
+// place of its U
+template <int VEC> struct SsdVec;
+template <> struct SsdVec<1> { using T = float; };
+template <> struct SsdVec<4> { using T = float4; };
+__device__ __forceinline__ float ssd_next(float S, float d, float u) { return fmaf(d, S, u); }
+__device__ __forceinline__ float4 ssd_next(float4 S, float d, float4 u) {
+    return make_float4(fmaf(d, S.x, u.x), fmaf(d, S.y, u.y), fmaf(d, S.z, u.z), fmaf(d, S.w, u.w));
+}
+
+template <int VEC>
+__global__ void __launch_bounds__(128) ssd_carry_kernel(const SS a) {
+    using V = typename SsdVec<VEC>::T;
+    const int e = blockIdx.x, h = blockIdx.y, i = blockIdx.z * blockDim.x + threadIdx.x, per = a.n_state * a.vdim / VEC;
     if (i >= per) return;
     const int row_e = a.ent_row[e], n = a.ent_len[e], b = a.slot[row_e], chunks = (n + kSsdChunk - 1) / kSsdChunk;
-    float* sp = a.state + ((size_t)b * a.heads + h) * per + i;
-    float S = a.pos[row_e] > 0 ? *sp : 0.f;
+    V* sp = reinterpret_cast<V*>(a.state) + ((size_t)b * a.heads + h) * per + i;
+    V S{};
+    if (a.pos[row_e] > 0) S = *sp;
     const size_t first = (size_t)(row_e / kSsdChunk + e), step = (size_t)a.heads * per;
-    float* U = a.chunk_state + (first * a.heads + h) * per + i;
+    V* U = reinterpret_cast<V*>(a.chunk_state) + (first * a.heads + h) * per + i;
     const float* dec = a.chunk_decay + first * a.heads + h;
-    for (int c0 = 0; c0 < chunks; c0 += 8) {   // eight loads in flight, then the dependent chain
-        float u[8], d[8];
+    constexpr int F = 8;
+    for (int c0 = 0; c0 < chunks; c0 += F) {   // F loads in flight, then the dependent chain
+        V u[F];
+        float d[F];
 #pragma unroll
-        for (int k = 0; k < 8; ++k) {
-            u[k] = c0 + k < chunks ? U[(size_t)(c0 + k) * step] : 0.f;
-            d[k] = c0 + k < chunks ? dec[(size_t)(c0 + k) * a.heads] : 0.f;
-        }
+        for (int k = 0; k < F; ++k)
+            if (c0 + k < chunks) {
+                u[k] = U[(size_t)(c0 + k) * step];
+                d[k] = dec[(size_t)(c0 + k) * a.heads];
+            }
 #pragma unroll
-        for (int k = 0; k < 8; ++k)
+        for (int k = 0; k < F; ++k)
             if (c0 + k < chunks) {
                 U[(size_t)(c0 + k) * step] = S;
-                S = fmaf(d[k], S, u[k]);
+                S = ssd_next(S, d[k], u[k]);
             }
     }
     *sp = S;
@@ -305,16 +330,18 @@ __global__ void __launch_bounds__(128) ssd_out_kernel(const SS a) {
     float* Cs = Ms + kSsdChunk * kSsdMs;          // [64][st]
     float* Ss = Cs + kSsdChunk * st;              // [npad][kSsdXs]
     const int cols = min(kSsdCols, P - p0);
-    ssd_chunk_sums(a, h, ck.row0, ck.len, dts, cum);
     const float* row = a.u + (size_t)ck.row0 * a.ld_u;
     ssd_stage(Cs, st, row + a.c_off + g * N, a.ld_u, kSsdChunk, ck.len, N, npad);
     ssd_stage(Xs, kSsdXs, row + a.x_off + h * P + p0, a.ld_u, kSsdChunk, ck.len, cols, kSsdCols);
     ssd_stage(Ss, kSsdXs, a.chunk_state + (((size_t)ck.place * a.heads + h) * N) * P + p0, P, npad, N, cols, kSsdCols);
-    __syncthreads();
-    const float* cb = a.chunk_cb + ((size_t)ck.place * a.groups + g) * kSsdChunk * kSsdChunk;
+    ssd_stage(Ms, kSsdMs, a.chunk_cb + ((size_t)ck.place * a.groups + g) * kSsdChunk * kSsdChunk, kSsdChunk, kSsdChunk, kSsdChunk, kSsdChunk, kSsdChunk);
+    ssd_chunk_sums(a, h, ck.row0, ck.len, dts, cum);
+    ssd_landed();
+#pragma unroll 4
     for (int i = threadIdx.x; i < kSsdChunk * kSsdChunk; i += 128) {
         const int r = i / kSsdChunk, j = i % kSsdChunk;
-        Ms[r * kSsdMs + j] = j <= r ? ssd_tf32(cb[i] * expf((float)(cum[r] - cum[j])) * dts[j]) : 0.f;
+        float* v = Ms + r * kSsdMs + j;
+        *v = j <= r ? ssd_tf32(*v * expf((float)(cum[r] - cum[j])) * dts[j]) : 0.f;
     }
     __syncthreads();
     const int warp = threadIdx.x / 32, lane = threadIdx.x % 32, gid = lane >> 2, tig = lane & 3, m0 = warp * 16;
@@ -323,20 +350,20 @@ __global__ void __launch_bounds__(128) ssd_out_kernel(const SS a) {
     for (int nt = 0; nt < 8; ++nt) acc[nt][0] = acc[nt][1] = acc[nt][2] = acc[nt][3] = 0.f;
     for (int k0 = 0; k0 < npad; k0 += 8) {   // what older chunks left
         const float* ar = Cs + (m0 + gid) * st + k0 + tig;
-        const float av[4] = {ar[0], ar[8 * st], ar[4], ar[8 * st + 4]};
+        const float av[4] = {ssd_tf32(ar[0]), ssd_tf32(ar[8 * st]), ssd_tf32(ar[4]), ssd_tf32(ar[8 * st + 4])};
         const float* br = Ss + (k0 + tig) * kSsdXs + gid;
 #pragma unroll
-        for (int nt = 0; nt < 8; ++nt) ssd_mma(acc[nt], av, br[nt * 8], br[4 * kSsdXs + nt * 8]);
+        for (int nt = 0; nt < 8; ++nt) ssd_mma(acc[nt], av, ssd_tf32(br[nt * 8]), ssd_tf32(br[4 * kSsdXs + nt * 8]));
     }
     const float e_lo = expf((float)cum[m0 + gid]), e_hi = expf((float)cum[m0 + gid + 8]);
 #pragma unroll
     for (int nt = 0; nt < 8; ++nt) { acc[nt][0] *= e_lo; acc[nt][1] *= e_lo; acc[nt][2] *= e_hi; acc[nt][3] *= e_hi; }
     for (int k0 = 0; k0 < m0 + 16; k0 += 8) {   // this chunk's own tokens, up to the warp's last row
         const float* ar = Ms + (m0 + gid) * kSsdMs + k0 + tig;
-        const float av[4] = {ar[0], ar[8 * kSsdMs], ar[4], ar[8 * kSsdMs + 4]};
+        const float av[4] = {ar[0], ar[8 * kSsdMs], ar[4], ar[8 * kSsdMs + 4]};   // rounded above
         const float* br = Xs + (k0 + tig) * kSsdXs + gid;
 #pragma unroll
-        for (int nt = 0; nt < 8; ++nt) ssd_mma(acc[nt], av, br[nt * 8], br[4 * kSsdXs + nt * 8]);
+        for (int nt = 0; nt < 8; ++nt) ssd_mma(acc[nt], av, ssd_tf32(br[nt * 8]), ssd_tf32(br[4 * kSsdXs + nt * 8]));
     }
     const float Dh = a.D[h];
 #pragma unroll
@@ -346,7 +373,7 @@ __global__ void __launch_bounds__(128) ssd_out_kernel(const SS a) {
             const int i = m0 + gid + (k >> 1) * 8, p = nt * 8 + tig * 2 + (k & 1);
             if (i < ck.len && p < cols)
                 a.out[(size_t)(ck.row0 + i) * ((size_t)a.heads * P) + h * P + p0 + p] =
-                    fmaf(Dh, row[(size_t)i * a.ld_u + a.x_off + h * P + p0 + p], acc[nt][k]);
+                    fmaf(Dh, Xs[i * kSsdXs + p], acc[nt][k]);
         }
 }
 
@@ -373,6 +400,55 @@ __global__ void __launch_bounds__(128) gated_group_rms_kernel(const float* __res
     const float rinv = 1.0f / sqrtf((red[0] + red[1] + red[2] + red[3]) / (float)per + eps);
     T* dst = out + t * n + c0;
     for (int i = threadIdx.x; i < per; i += 128) dst[i] = DT<T>::from_f(vs[i] * rinv * w[c0 + i]);
+}
+
+// the same for parts of at most 16 * THREADS columns in whole groups of four: everything is loaded up front and lives in registers
+template <typename T, int THREADS>
+__global__ void __launch_bounds__(THREADS) gated_group_rms_reg_kernel(const float* __restrict__ y, const float* __restrict__ z, long long ld_z,
+                                                                      const float* __restrict__ w, T* __restrict__ out, int n, int per, float eps) {
+    __shared__ float red[THREADS / 32];
+    const size_t t = blockIdx.x;
+    const int c0 = blockIdx.y * per;
+    const float* yr = y + t * n + c0;
+    const float* zr = z + t * ld_z + c0;
+    float4 v[4], g[4], w4[4];
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+        const int i = 4 * (threadIdx.x + THREADS * k);
+        v[k] = g[k] = w4[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (i < per) {
+            v[k] = *reinterpret_cast<const float4*>(yr + i);
+            g[k] = *reinterpret_cast<const float4*>(zr + i);
+            w4[k] = *reinterpret_cast<const float4*>(w + c0 + i);
+        }
+    }
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+        v[k].x *= g[k].x / (1.f + expf(-g[k].x)); v[k].y *= g[k].y / (1.f + expf(-g[k].y));
+        v[k].z *= g[k].z / (1.f + expf(-g[k].z)); v[k].w *= g[k].w / (1.f + expf(-g[k].w));
+        ss += v[k].x * v[k].x + v[k].y * v[k].y + v[k].z * v[k].z + v[k].w * v[k].w;
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    if (threadIdx.x % 32 == 0) red[threadIdx.x / 32] = ss;
+    __syncthreads();
+    float tot = 0.f;
+#pragma unroll
+    for (int k = 0; k < THREADS / 32; ++k) tot += red[k];
+    const float r = 1.0f / sqrtf(tot / (float)per + eps);
+    T* dst = out + t * n + c0;
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+        const int i = 4 * (threadIdx.x + THREADS * k);
+        if (i >= per) continue;
+        const float f[4] = {v[k].x * r * w4[k].x, v[k].y * r * w4[k].y, v[k].z * r * w4[k].z, v[k].w * r * w4[k].w};
+        if constexpr (sizeof(T) == 4) *reinterpret_cast<float4*>(dst + i) = make_float4(f[0], f[1], f[2], f[3]);
+        else {
+            const __nv_bfloat162 lo = __floats2bfloat162_rn(f[0], f[1]), hi = __floats2bfloat162_rn(f[2], f[3]);
+            *reinterpret_cast<uint2*>(dst + i) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+        }
+    }
 }
 
 static size_t ssd_places(int n_tokens, int n_entries) { return (size_t)n_tokens / kSsdChunk + (size_t)n_entries + 1; }
@@ -430,8 +506,11 @@ extern "C" int b200_ssd_scan(const b200_ssd_scan_args* p, void* stream) {
         ssd_cb_kernel<<<dim3(p->n_entries, chunks, p->groups), 128, sm_cb, s>>>(a);
         const dim3 grid(p->n_entries * a.col_blocks, chunks, p->heads);
         ssd_state_kernel<<<grid, 128, sm_st, s>>>(a);
-        const int per = p->n_state * p->vdim;
-        ssd_carry_kernel<<<dim3(p->n_entries, p->heads, (per + 255) / 256), 256, 0, s>>>(a);
+        const int per = p->n_state * p->vdim;   // a head's state starts on a multiple of `per` floats
+        if (per % 4 == 0 && (reinterpret_cast<uintptr_t>(p->state) & 15u) == 0)
+            ssd_carry_kernel<4><<<dim3(p->n_entries, p->heads, (per / 4 + 127) / 128), 128, 0, s>>>(a);
+        else
+            ssd_carry_kernel<1><<<dim3(p->n_entries, p->heads, (per + 127) / 128), 128, 0, s>>>(a);
         ssd_out_kernel<<<grid, 128, sm_out, s>>>(a);
         count_launch(4);
         return (int)cudaGetLastError();
@@ -447,6 +526,20 @@ extern "C" int b200_gated_group_rms(const float* y, const float* z, long long ld
     if (smem > 200 * 1024 || parts > 65535) return B200_EUNSUPPORTED;
     const dim3 grid(n_tokens, parts);
     cudaStream_t s = (cudaStream_t)stream;
+    const int per = n / parts;
+    auto al16 = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15u) == 0; };
+    if (per % 4 == 0 && per <= 16 * 512 && ld_z % 4 == 0 && al16(y) && al16(z) && al16(w) && al16(out) && (out_dtype == B200_BF16 || out_dtype == B200_F32)) {
+        const bool bf = out_dtype == B200_BF16;
+        if (per <= 16 * 128) {
+            if (bf) gated_group_rms_reg_kernel<__nv_bfloat16, 128><<<grid, 128, 0, s>>>(y, z, ld_z, w, (__nv_bfloat16*)out, n, per, eps);
+            else gated_group_rms_reg_kernel<float, 128><<<grid, 128, 0, s>>>(y, z, ld_z, w, (float*)out, n, per, eps);
+        } else {
+            if (bf) gated_group_rms_reg_kernel<__nv_bfloat16, 512><<<grid, 512, 0, s>>>(y, z, ld_z, w, (__nv_bfloat16*)out, n, per, eps);
+            else gated_group_rms_reg_kernel<float, 512><<<grid, 512, 0, s>>>(y, z, ld_z, w, (float*)out, n, per, eps);
+        }
+        count_launch();
+        return (int)cudaGetLastError();
+    }
     if (out_dtype == B200_BF16) {
         static unsigned long long done = 0;
         if (smem > 48 * 1024) ensure_max_dynamic_smem((const void*)gated_group_rms_kernel<__nv_bfloat16>, 200 * 1024, done);

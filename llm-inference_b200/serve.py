@@ -528,3 +528,61 @@ def random_sakevik(width, vocab, layers, buckets=65521, seed=0):
             w[pre + "mlp.gate"], w[pre + "mlp.up"], w[pre + "mlp.down"] = rnd(f, width), rnd(f, width), rnd(width, f)
         cfg["layers"].append(dict(type=sp["type"], mixer=mx, mlp=ml))
     return cfg, w
+
+
+def random_filipel(width, vocab, layers, seed=0):
+    """(config, tensors) of a random Filipel model. layers: dicts with type 'latent_attention' (heads, dim, rot_dim, vdim, q_rank,
+    kv_rank, optionally kv_from) | 'parallel' (left = dict(heads, kv_heads, dim, vdim, window), right = dict(heads, vdim, state,
+    groups, conv, norm_groups)); ff = None | int (dense) | (ff, experts, top, groups, keep)"""
+    import math
+
+    import torch
+
+    g = torch.Generator().manual_seed(seed)
+
+    def rnd(*shape, s=None):
+        return (torch.randn(*shape, generator=g) * (s if s is not None else 1.0 / math.sqrt(shape[-1]))).to(torch.bfloat16)
+
+    cfg = dict(architecture="Filipel", vocab=vocab, width=width, norm=dict(eps=1e-6), residual_mult=0.7, layers=[])
+    w = {"embed": rnd(vocab, width, s=1.0), "head": rnd(vocab, width), "final.norm": torch.ones(width)}
+    for i, sp in enumerate(layers):
+        pre, mp = f"l{i}.", f"l{i}.mix."
+        w[pre + "norm1"] = torch.ones(width)
+        if sp["type"] == "latent_attention":
+            H, d, dr, dv, Q, R = sp["heads"], sp["dim"], sp["rot_dim"], sp["vdim"], sp["q_rank"], sp["kv_rank"]
+            mx = dict(heads=H, dim=d, rot_dim=dr, vdim=dv, q_rank=Q, kv_rank=R, scale=1.0 / math.sqrt(d + dr), rot=dict(base=500000.0, dims=dr))
+            if sp.get("kv_from") is not None:
+                mx["kv_from"] = sp["kv_from"]
+            else:
+                w[mp + "dkv"], w[mp + "dkv.norm"] = rnd(R + dr, width), torch.ones(R)
+            w[mp + "dq"], w[mp + "dq.norm"], w[mp + "uq"] = rnd(Q, width), torch.ones(Q), rnd(H * (d + dr), Q)
+            w[mp + "uk"], w[mp + "uv"] = rnd(H * d, R), rnd(H * dv, R)
+            w[mp + "g"], w[mp + "o"] = rnd(H * dv, width), rnd(width, H * dv)
+        else:
+            a, b, lp, rp = sp["left"], sp["right"], mp + "left.", mp + "right."
+            H, G, d, dv = a["heads"], a["kv_heads"], a["dim"], a["vdim"]
+            w[lp + "q"], w[lp + "k"], w[lp + "v"] = rnd(H * d, width), rnd(G * d, width), rnd(G * dv, width)
+            w[lp + "temp"], w[lp + "talk"] = torch.ones(H), torch.eye(H) + rnd(H, H, s=0.3 / math.sqrt(H)).float()
+            w[lp + "g"], w[lp + "o"], w[lp + "out"] = rnd(H * dv, width), rnd(width, H * dv), torch.ones(width)
+            Hs, P, N, Gs, taps = b["heads"], b["vdim"], b["state"], b["groups"], b["conv"]
+            ch = Hs * P + 2 * Gs * N
+            w[rp + "in"], w[rp + "conv"], w[rp + "conv.b"] = rnd(Hs * P + ch + Hs, width), rnd(ch, taps, s=0.5), torch.zeros(ch)
+            w[rp + "dt_bias"], w[rp + "A_log"] = torch.full((Hs,), -3.0), torch.log(torch.linspace(1, 16, Hs))
+            w[rp + "D"], w[rp + "norm"], w[rp + "o"], w[rp + "out"] = torch.ones(Hs), torch.ones(Hs * P), rnd(width, Hs * P), torch.ones(width)
+            mx = dict(left=dict(heads=H, kv_heads=G, dim=d, vdim=dv, scale=1.0 / math.sqrt(d), rot=dict(base=10000.0, dims=d), mask=dict(size=a["window"])),
+                      right=dict(heads=Hs, vdim=P, state=N, groups=Gs, conv=taps, norm_groups=b["norm_groups"]))
+        ff = sp.get("ff")
+        if ff is None:
+            ml = None
+        elif isinstance(ff, int):
+            ml = dict(kind="dense", ff=ff)
+            w[pre + "mlp.up"], w[pre + "mlp.down"], w[pre + "mlp.act"] = rnd(ff, width), rnd(width, ff), torch.tensor([0.5, 0.3, 0.2, 0.0])
+        else:
+            f, E, top, gc, keep = ff
+            ml = dict(kind="moe", expert=dict(ff=f), router=dict(experts=E, top=top, groups=dict(count=gc, keep=keep)))
+            w[pre + "mlp.router"] = rnd(E, width)
+            for e in range(E):
+                p = pre + f"mlp.e{e}."
+                w[p + "gate"], w[p + "up"], w[p + "down"] = rnd(f, width), rnd(f, width), rnd(width, f)
+        cfg["layers"].append(dict(type=sp["type"], mixer=mx, mlp=ml))
+    return cfg, w
