@@ -19,7 +19,7 @@ def S(pkg):
 
 def test_registry_lists_the_families(S):
     fams = S.lib().b200_model_families().decode().split(",")
-    assert "Nekodra" in fams and "Musilorn" in fams and "Tomalix" in fams and "Sakevik" in fams and "llama" in fams
+    assert "Nekodra" in fams and "Musilorn" in fams and "Tomalix" in fams and "Sakevik" in fams and "Filipel" in fams and "llama" in fams
 
 
 def test_unknown_architecture_and_broken_config(S, tmp_path):
@@ -270,3 +270,122 @@ def test_sakevik_oracle_pieces_agree_with_closed_forms():
     assert float(y[2, 0]) == pytest.approx(2.0 / (1 + math.exp(-1.702 * 2.0)) * 3.0)
     assert float(y[1, 0]) == pytest.approx(0.5 / (1 + math.exp(-1.702 * 0.5)) * 1.5)
     assert float(y[0, 0]) == pytest.approx(-5.0 / (1 + math.exp(1.702 * 5.0)) * -1.0)
+
+
+def test_filipel_configuration_errors_end_before_any_cuda_call(S, tmp_path):
+    import json
+    lat = dict(type="latent_attention", mixer=dict(heads=2, dim=4, vdim=4, q_rank=5, kv_rank=6, rot_dim=4, scale=0.5, rot=dict(base=100.0, dims=4)), mlp=None)
+    par = dict(type="parallel", mixer=dict(left=dict(heads=4, kv_heads=2, dim=4, vdim=4, scale=0.5, rot=dict(base=10.0, dims=4), mask=dict(size=9)),
+                                           right=dict(heads=4, vdim=2, state=3, groups=2, conv=4, norm_groups=2)), mlp=None)
+    moe = dict(kind="moe", expert=dict(ff=8), router=dict(experts=6, top=2, groups=dict(count=3, keep=2)))
+
+    def refused(layers, text, **top):
+        cfg = dict(architecture="Filipel", width=8, vocab=5, norm=dict(eps=1e-5), residual_mult=0.5, layers=layers, **top)
+        (tmp_path / "config.json").write_text(json.dumps(cfg))
+        with pytest.raises(RuntimeError, match=text):
+            S.Model(tmp_path)
+
+    def mixer(base, **kw):
+        return dict(base, mixer=dict(base["mixer"], **kw))
+
+    def side(name, **kw):
+        return mixer(par, **{name: dict(par["mixer"][name], **kw)})
+
+    def router(**kw):
+        return dict(lat, mlp=dict(moe, router=dict(moe["router"], **kw)))
+    refused([], "required")
+    refused([dict(lat, type="retention")], "not part of this family")
+    refused([dict(lat, mixer=None)], "no mixer")
+    refused([dict(lat, mlp=dict(kind="glu", ff=8))], "feed-forward kind")
+    refused([dict(lat, mlp=dict(kind="dense"))], "mlp.ff")
+    refused([mixer(lat, q_rank=0)], "q_rank")
+    refused([mixer(lat, rot=dict(base=100.0, dims=2))], "rot_dim")
+    refused([mixer(lat, kv_rank=640)], "wider than 640")
+    refused([lat, mixer(lat, kv_from=1)], "kv_from")
+    refused([par, mixer(lat, kv_from=0)], "kv_from")
+    refused([lat, mixer(lat, kv_from=0), mixer(lat, kv_from=1)], "kv_from")
+    refused([lat, mixer(lat, kv_from=0, kv_rank=7)], "kv_from: kv_rank")
+    refused([lat, mixer(lat, kv_from=0, rot=dict(base=99.0, dims=4))], "kv_from: kv_rank, rot_dim and rotation")
+    refused([side("left", heads=3)], "multiple of kv_heads")
+    refused([side("left", rot=dict(base=10.0, dims=6))], "at most dim")
+    refused([side("left", mask=dict(size=0))], "mask.size")
+    refused([side("right", groups=3)], "multiple of groups")
+    refused([side("right", norm_groups=3)], "norm_groups")
+    refused([side("right", state=300)], "state above 256")
+    refused([mixer(par, right=None)], "left and right")
+    refused([router(top=7)], "router.top")
+    refused([router(groups=dict(count=4, keep=2))], "count must divide")
+    refused([router(top=5)], "kept groups must hold")
+
+
+def test_filipel_random_checkpoint_and_workspaces(S, tmp_path):
+    """the random checkpoint names what the loader asks for, and the workspace sizes follow the shape of the step"""
+    import json
+    par = dict(type="parallel", left=dict(heads=4, kv_heads=2, dim=8, vdim=8, window=9), right=dict(heads=4, vdim=16, state=8, groups=1, conv=4, norm_groups=1))
+    lat = dict(type="latent_attention", heads=2, dim=8, rot_dim=4, vdim=8, q_rank=12, kv_rank=16)
+    cfg, w = S.random_filipel(32, 50, [dict(lat, ff=24), dict(par, ff=(8, 4, 2, 2, 1)), dict(lat, kv_from=0, ff=None)])
+    S.write_checkpoint(tmp_path, cfg, w)
+    raw = (tmp_path / "model.safetensors").read_bytes()
+    header = json.loads(raw[8:8 + int.from_bytes(raw[:8], "little")])
+    assert header["l1.mix.right.in"]["shape"] == [64 + 64 + 16 + 4, 32] and header["l1.mix.left.talk"]["shape"] == [4, 4]
+    assert "l0.mix.dkv" in header and "l2.mix.dkv" not in header and header["l0.mlp.act"]["shape"] == [4]
+    assert header["l1.mlp.e3.down"]["shape"] == [32, 8] and "l2.mlp.up" not in header
+    L = S.lib()
+    assert L.b200_mixed_attention_workspace_bytes(1, 4, 9, 100) == 0                     # a single token needs none
+    few, many = L.b200_mixed_attention_workspace_bytes(100, 4, 9, 5000), L.b200_mixed_attention_workspace_bytes(100, 4, 0, 5000)
+    assert few == 128 * (4 * 192 * 6 + 4 * 8 + 8) and many > 20 * few                     # 9 + 126 columns in whole tiles; no window: all
+    assert L.b200_mixed_attention_workspace_bytes(1 << 20, 16, 1024, 1 << 20) <= 256 << 20   # long prompts go block by block
+    assert L.b200_ssd_scan_workspace_bytes(127, 1, 4, 1, 16, 8) == 0 and L.b200_ssd_scan_workspace_bytes(128, 1, 4, 1, 16, 8) >= 4 * 4 * 16 * 8 * 4
+
+
+def test_filipel_oracle_pieces_agree_with_closed_forms():
+    """the plain implementation of the fifth family: both norms, the window, the mix, the recurrence against its unrolled sum, the
+    convolution, the normed powers, the router's groups"""
+    import filipel_oracle as K
+    g = torch.Generator().manual_seed(3)
+    D = torch.float64
+    x = torch.randn(4, 6, generator=g, dtype=D)
+    n = K.layer_norm(x, torch.full((6,), 2.0, dtype=D), 0.0)
+    assert torch.allclose(n.mean(-1), torch.zeros(4, dtype=D), atol=1e-12) and torch.allclose(n.pow(2).mean(-1), torch.full((4,), 4.0, dtype=D))
+    assert torch.allclose(K.rms_norm(x, torch.ones(6, dtype=D), 0.0).pow(2).mean(-1), torch.ones(4, dtype=D))
+    m = K.visible(6, 3)
+    assert m[5].tolist() == [False, False, False, True, True, True] and m[1].tolist() == [True, True, False, False, False, False]
+    assert K.visible(3, 0).tolist() == [[True, False, False], [True, True, False], [True, True, True]]
+    q = torch.randn(5, 2, 6, generator=g, dtype=D)
+    r = K.turn_half(q, dict(base=100.0, dims=4))
+    a = 3 * 100.0 ** (-2 / 4)
+    assert torch.equal(r[..., 4:], q[..., 4:]) and torch.equal(r[0], q[0])
+    assert torch.allclose(r[3, 1, 1], q[3, 1, 1] * math.cos(a) - q[3, 1, 3] * math.sin(a))
+    assert torch.allclose(r[3, 1, 3], q[3, 1, 3] * math.cos(a) + q[3, 1, 1] * math.sin(a))
+    # two heads, two positions, zero queries: every weight of position 1 is a half; the mix acts on the heads
+    talk = torch.tensor([[1.0, 2.0], [0.0, -1.0]], dtype=D)
+    v = torch.tensor([[[1.0]], [[3.0]]], dtype=D)
+    o = K.mixed_attention(torch.zeros(2, 2, 1, dtype=D), torch.zeros(2, 1, 1, dtype=D), v, 1.0, torch.ones(2, dtype=D), talk, 0)
+    assert torch.allclose(o[:, :, 0], torch.tensor([[3.0, -1.0], [6.0, -2.0]], dtype=D))
+    o = K.mixed_attention(torch.zeros(2, 2, 1, dtype=D), torch.zeros(2, 1, 1, dtype=D), v, 1.0, torch.ones(2, dtype=D), talk, 1)
+    assert torch.allclose(o[1, :, 0], torch.tensor([9.0, -3.0], dtype=D))
+    # temperature: ln 3 times the score difference of one
+    o = K.mixed_attention(torch.ones(2, 1, 1, dtype=D), torch.tensor([[[0.0]], [[1.0]]], dtype=D), v, 1.0, torch.tensor([math.log(3.0)], dtype=D),
+                          torch.ones(1, 1, dtype=D), 0)
+    assert float(o[1, 0, 0]) == pytest.approx(0.25 * 1 + 0.75 * 3)
+    # one head, one state, one column: the output is a sum over older inputs, each decayed by every later step
+    B, Cc, xs, dt = (torch.rand(5, generator=g, dtype=D) for _ in range(4))
+    y = K.ssd(xs.view(5, 1, 1), B.view(5, 1, 1), Cc.view(5, 1, 1), dt.view(5, 1), torch.tensor([0.4], dtype=D), torch.tensor([0.7], dtype=D))
+    for t in range(5):
+        want = 0.7 * xs[t] + sum(Cc[t] * B[j] * dt[j] * xs[j] * math.exp(-math.exp(0.4) * float(dt[j + 1:t + 1].sum())) for j in range(t + 1))
+        assert float(y[t, 0, 0]) == pytest.approx(float(want))
+    u = torch.tensor([[1.0], [2.0], [4.0]], dtype=D)
+    c = K.causal_conv_silu(u, torch.tensor([[10.0, 1.0]], dtype=D), torch.tensor([0.5], dtype=D))
+    assert torch.allclose(c[:, 0], K.silu(torch.tensor([1.5, 12.5, 24.5], dtype=D)))
+    z = torch.tensor([[1.0, -2.0]], dtype=D)
+    p = K.poly_norm(z, (1.0, 0.5, 2.0, 0.25), 0.0)
+    want = [s / math.sqrt(2.5) + 0.5 * s * s / math.sqrt(8.5) + 2 * s ** 3 / math.sqrt(32.5) + 0.25 for s in (1.0, -2.0)]
+    assert p[0].tolist() == pytest.approx(want)
+    # the second largest logit lies in a group that is not kept
+    logits = torch.log(torch.tensor([[8.0, 1.0, 7.0, 0.5, 6.0, 5.0]], dtype=D))
+    chosen, w = K.route(logits, dict(count=3, keep=1), 2)
+    assert chosen.tolist() == [[0, 1]] and w[0].tolist() == pytest.approx([8 / 9, 1 / 9])
+    chosen, w = K.route(logits, None, 2)
+    assert chosen.tolist() == [[0, 2]] and w[0].tolist() == pytest.approx([8 / 15, 7 / 15])
+    gn = K.gated_group_norm(torch.ones(1, 4, dtype=D), torch.tensor([[1.0, 1.0, 5.0, 5.0]], dtype=D), torch.tensor([1.0, 2.0, 3.0, 4.0], dtype=D), 2, 0.0)
+    assert torch.allclose(gn, torch.tensor([[1.0, 2.0, 3.0, 4.0]], dtype=D))
