@@ -8,7 +8,7 @@
 
 namespace b200 {
 
-constexpr int kPrPer = 8, kPrMaxTop = 16;
+constexpr int kPrMaxTop = 16;
 
 // sums of two values over a CTA, the same order in every thread
 template <int THREADS>
@@ -27,8 +27,8 @@ __device__ __forceinline__ float2 block_sum2(float a, float b, float2* red) {
     return s;
 }
 
-// rows of at most THREADS * kPrPer values: every operand of the row is loaded up front and lives in registers
-template <typename T, int THREADS>
+// rows of at most THREADS * PER values: every operand of the row is loaded up front and lives in registers
+template <typename T, int THREADS, int PER>
 __global__ void __launch_bounds__(THREADS) parallel_residual_reg_kernel(const b200_parallel_residual_args a) {
     __shared__ float2 red[THREADS / 32];
     __shared__ int e_dest[kPrMaxTop];
@@ -42,9 +42,9 @@ __global__ void __launch_bounds__(THREADS) parallel_residual_reg_kernel(const b2
         }
         __syncthreads();
     }
-    float v[kPrPer], p1[kPrPer], p2[kPrPer], p3[kPrPer], w1[kPrPer], w2[kPrPer], lw[kPrPer], lb[kPrPer];
+    float v[PER], p1[PER], p2[PER], p3[PER], w1[PER], w2[PER], lw[PER], lb[PER];
 #pragma unroll
-    for (int k = 0; k < kPrPer; ++k) {
+    for (int k = 0; k < PER; ++k) {
         const int c = threadIdx.x + THREADS * k;
         const bool in = c < width;
         v[k] = in ? a.x[base + c] : 0.f;
@@ -62,25 +62,25 @@ __global__ void __launch_bounds__(THREADS) parallel_residual_reg_kernel(const b2
             const int d = e_dest[j];
             if (d < 0) continue;
             const float* er = a.expert_out + (size_t)d * width;
-            float e[kPrPer];
+            float e[PER];
 #pragma unroll
-            for (int k = 0; k < kPrPer; ++k) e[k] = threadIdx.x + THREADS * k < width ? er[threadIdx.x + THREADS * k] : 0.f;
+            for (int k = 0; k < PER; ++k) e[k] = threadIdx.x + THREADS * k < width ? er[threadIdx.x + THREADS * k] : 0.f;
 #pragma unroll
-            for (int k = 0; k < kPrPer; ++k) p3[k] = fmaf(e_w[j], e[k], p3[k]);
+            for (int k = 0; k < PER; ++k) p3[k] = fmaf(e_w[j], e[k], p3[k]);
         }
     }
     float r1 = 1.f, r2 = 1.f;
     if (a.w1 || a.w2) {
         float s1 = 0.f, s2 = 0.f;
 #pragma unroll
-        for (int k = 0; k < kPrPer; ++k) { s1 += p1[k] * p1[k]; s2 += p2[k] * p2[k]; }
+        for (int k = 0; k < PER; ++k) { s1 += p1[k] * p1[k]; s2 += p2[k] * p2[k]; }
         const float2 s = block_sum2<THREADS>(s1, s2, red);
         r1 = a.w1 ? 1.0f / sqrtf(s.x / (float)width + a.eps) : 1.f;
         r2 = a.w2 ? 1.0f / sqrtf(s.y / (float)width + a.eps) : 1.f;
     }
     float sum = 0.f;
 #pragma unroll
-    for (int k = 0; k < kPrPer; ++k) {
+    for (int k = 0; k < PER; ++k) {
         const int c = threadIdx.x + THREADS * k;
         if (c < width) {
             float y = 0.f;
@@ -96,14 +96,14 @@ __global__ void __launch_bounds__(THREADS) parallel_residual_reg_kernel(const b2
     const float mean = block_sum2<THREADS>(sum, 0.f, red).x / (float)width;
     float q = 0.f;
 #pragma unroll
-    for (int k = 0; k < kPrPer; ++k) {
+    for (int k = 0; k < PER; ++k) {
         const float d = threadIdx.x + THREADS * k < width ? v[k] - mean : 0.f;
         q += d * d;
     }
     const float rstd = 1.0f / sqrtf(block_sum2<THREADS>(q, 0.f, red).x / (float)width + a.eps);
     T* out = reinterpret_cast<T*>(a.out) + base;
 #pragma unroll
-    for (int k = 0; k < kPrPer; ++k) {
+    for (int k = 0; k < PER; ++k) {
         const int c = threadIdx.x + THREADS * k;
         if (c < width) out[c] = DT<T>::from_f((v[k] - mean) * rstd * lw[k] + lb[k]);
     }
@@ -158,8 +158,9 @@ __global__ void __launch_bounds__(256) parallel_residual_kernel(const b200_paral
 
 template <typename T>
 static void launch_pr(const b200_parallel_residual_args& a, size_t smem, cudaStream_t s) {
-    if (a.width <= 256 * kPrPer) parallel_residual_reg_kernel<T, 256><<<a.n_rows, 256, 0, s>>>(a);
-    else if (a.width <= 1024 * kPrPer) parallel_residual_reg_kernel<T, 1024><<<a.n_rows, 1024, 0, s>>>(a);
+    if (a.width <= 512) parallel_residual_reg_kernel<T, 128, 4><<<a.n_rows, 128, 0, s>>>(a);
+    else if (a.width <= 2048) parallel_residual_reg_kernel<T, 512, 4><<<a.n_rows, 512, 0, s>>>(a);
+    else if (a.width <= 4096) parallel_residual_reg_kernel<T, 1024, 4><<<a.n_rows, 1024, 0, s>>>(a);
     else {
         static unsigned long long done = 0;
         if (smem > 48 * 1024) ensure_max_dynamic_smem((const void*)parallel_residual_kernel<T>, 200 * 1024, done);

@@ -317,7 +317,7 @@ __global__ void __launch_bounds__(128) ssd_carry_kernel(const SS a) {
     *sp = S;
 }
 
-__global__ void __launch_bounds__(128) ssd_out_kernel(const SS a) {
+__global__ void __launch_bounds__(256) ssd_out_kernel(const SS a) {
     extern __shared__ __align__(16) float sm[];
     __shared__ double cum[kSsdChunk];
     __shared__ float dts[kSsdChunk];
@@ -338,39 +338,40 @@ __global__ void __launch_bounds__(128) ssd_out_kernel(const SS a) {
     ssd_chunk_sums(a, h, ck.row0, ck.len, dts, cum);
     ssd_landed();
 #pragma unroll 4
-    for (int i = threadIdx.x; i < kSsdChunk * kSsdChunk; i += 128) {
+    for (int i = threadIdx.x; i < kSsdChunk * kSsdChunk; i += 256) {
         const int r = i / kSsdChunk, j = i % kSsdChunk;
         float* v = Ms + r * kSsdMs + j;
         *v = j <= r ? ssd_tf32(*v * expf((float)(cum[r] - cum[j])) * dts[j]) : 0.f;
     }
     __syncthreads();
-    const int warp = threadIdx.x / 32, lane = threadIdx.x % 32, gid = lane >> 2, tig = lane & 3, m0 = warp * 16;
-    float acc[8][4];
+    const int warp = threadIdx.x / 32, lane = threadIdx.x % 32, gid = lane >> 2, tig = lane & 3;
+    const int m0 = (warp & 3) * 16, q0 = (warp >> 2) * 32;   // eight warps: 16 rows x 32 value columns each
+    float acc[4][4];
 #pragma unroll
-    for (int nt = 0; nt < 8; ++nt) acc[nt][0] = acc[nt][1] = acc[nt][2] = acc[nt][3] = 0.f;
+    for (int nt = 0; nt < 4; ++nt) acc[nt][0] = acc[nt][1] = acc[nt][2] = acc[nt][3] = 0.f;
     for (int k0 = 0; k0 < npad; k0 += 8) {   // what older chunks left
         const float* ar = Cs + (m0 + gid) * st + k0 + tig;
         const float av[4] = {ssd_tf32(ar[0]), ssd_tf32(ar[8 * st]), ssd_tf32(ar[4]), ssd_tf32(ar[8 * st + 4])};
-        const float* br = Ss + (k0 + tig) * kSsdXs + gid;
+        const float* br = Ss + (k0 + tig) * kSsdXs + q0 + gid;
 #pragma unroll
-        for (int nt = 0; nt < 8; ++nt) ssd_mma(acc[nt], av, ssd_tf32(br[nt * 8]), ssd_tf32(br[4 * kSsdXs + nt * 8]));
+        for (int nt = 0; nt < 4; ++nt) ssd_mma(acc[nt], av, ssd_tf32(br[nt * 8]), ssd_tf32(br[4 * kSsdXs + nt * 8]));
     }
     const float e_lo = expf((float)cum[m0 + gid]), e_hi = expf((float)cum[m0 + gid + 8]);
 #pragma unroll
-    for (int nt = 0; nt < 8; ++nt) { acc[nt][0] *= e_lo; acc[nt][1] *= e_lo; acc[nt][2] *= e_hi; acc[nt][3] *= e_hi; }
+    for (int nt = 0; nt < 4; ++nt) { acc[nt][0] *= e_lo; acc[nt][1] *= e_lo; acc[nt][2] *= e_hi; acc[nt][3] *= e_hi; }
     for (int k0 = 0; k0 < m0 + 16; k0 += 8) {   // this chunk's own tokens, up to the warp's last row
         const float* ar = Ms + (m0 + gid) * kSsdMs + k0 + tig;
         const float av[4] = {ar[0], ar[8 * kSsdMs], ar[4], ar[8 * kSsdMs + 4]};   // rounded above
-        const float* br = Xs + (k0 + tig) * kSsdXs + gid;
+        const float* br = Xs + (k0 + tig) * kSsdXs + q0 + gid;
 #pragma unroll
-        for (int nt = 0; nt < 8; ++nt) ssd_mma(acc[nt], av, ssd_tf32(br[nt * 8]), ssd_tf32(br[4 * kSsdXs + nt * 8]));
+        for (int nt = 0; nt < 4; ++nt) ssd_mma(acc[nt], av, ssd_tf32(br[nt * 8]), ssd_tf32(br[4 * kSsdXs + nt * 8]));
     }
     const float Dh = a.D[h];
 #pragma unroll
-    for (int nt = 0; nt < 8; ++nt)
+    for (int nt = 0; nt < 4; ++nt)
 #pragma unroll
         for (int k = 0; k < 4; ++k) {
-            const int i = m0 + gid + (k >> 1) * 8, p = nt * 8 + tig * 2 + (k & 1);
+            const int i = m0 + gid + (k >> 1) * 8, p = q0 + nt * 8 + tig * 2 + (k & 1);
             if (i < ck.len && p < cols)
                 a.out[(size_t)(ck.row0 + i) * ((size_t)a.heads * P) + h * P + p0 + p] =
                     fmaf(Dh, Xs[i * kSsdXs + p], acc[nt][k]);
@@ -511,7 +512,7 @@ extern "C" int b200_ssd_scan(const b200_ssd_scan_args* p, void* stream) {
             ssd_carry_kernel<4><<<dim3(p->n_entries, p->heads, (per / 4 + 127) / 128), 128, 0, s>>>(a);
         else
             ssd_carry_kernel<1><<<dim3(p->n_entries, p->heads, (per + 127) / 128), 128, 0, s>>>(a);
-        ssd_out_kernel<<<grid, 128, sm_out, s>>>(a);
+        ssd_out_kernel<<<grid, 256, sm_out, s>>>(a);
         count_launch(4);
         return (int)cudaGetLastError();
     }
