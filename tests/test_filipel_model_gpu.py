@@ -29,7 +29,7 @@ SHAPES = {
     # beside pages of 64; experts in groups
     "mix": dict(width=48, vocab=61, mult=0.6, layers=[
         lat(4, 8, 4, 12, 20, 24, base=50.0, ff=40),
-        par((4, 2, 16, 8, 37, dict(rot_dims=8, base=100.0)), (4, 6, 10, 2, 4, 2), ff=(16, 12, 4, 4, 3)),
+        par((4, 2, 16, 8, 37, dict(rot_dims=8, base=100.0)), (4, 6, 10, 2, 4, 2), ff=(16, 10, 3, 5, 3)),
         lat(6, 4, 4, 6, 12, 24, base=50.0, scale=0.4, kv_from=0, ff=None),
         par((2, 1, 8, 12, 21, dict(base=30.0)), (2, 12, 7, 1, 3, 1), ff=24),
         lat(4, 8, 6, 8, 9, 16, base=200.0, ff=(12, 6, 2, 3, 1))]),
