@@ -14,6 +14,8 @@
  * weights, rotated values and head gates, or of windowed latent attention with a shared rotary key part; clamped gated
  * feed-forwards), "Filipel" (parallel layers of latent attention with low-rank queries, or of windowed attention whose weights
  * are mixed across heads beside a state-space recurrence; routed experts in groups, a dense feed-forward of normed powers),
+ * "Mazotar" (several residual streams with learned connections; attention with a distance bias and a learned sink, of its own or on an
+ * earlier layer's keys, or an mLSTM matrix memory; routed experts whose weight multiplies their input, beside a gated shared one),
  * "llama" (the reference's weight directory, llama_weights.cc:41-53, with
  * a config.json naming the b200_model_config fields).
  */
@@ -68,6 +70,7 @@ typedef struct b200_gemm_grouped_args {
     int epi;
     int a_dtype, w_dtype, c_dtype;   /* B200_F32 / B200_BF16                                                   */
     float epi_param;           /* B200_GG_GLU_CLAMP: the limit                                                   */
+    const float* row_scale;    /* fp32 [rows] or NULL: row r of A counts times row_scale[r] (applied to the products) */
 } b200_gemm_grouped_args;
 int b200_gemm_grouped(const b200_gemm_grouped_args* args, void* stream);
 
@@ -160,11 +163,21 @@ int b200_moe_route_logits(const void* h, int h_dtype, const float* w_router, con
  * n_out must be a multiple of groups and top at most keep * n_out / groups. groups 1: no restriction. */
 int b200_moe_route_groups(const void* h, int h_dtype, const float* w_router, int n_tokens, int width, int n_out, int top,
                           int groups, int keep, int* chosen, float* weight, void* stream);
+/* Router whose weights are sigmoids of its own: z = h W_r^T (fp32 accumulate; w_router fp32 [n_out + n_gates, width]); the `top`
+ * largest z of the first n_out are chosen (ties: the lower index), their weights are sigmoid(z), not renormalised; gates
+ * [n_tokens, n_gates] (may be NULL with n_gates 0) receives the sigmoids of the remaining rows (gates of shared experts). */
+int b200_moe_route_sigmoid(const void* h, int h_dtype, const float* w_router, int n_tokens, int width, int n_out, int top, int n_gates,
+                           int* chosen, float* weight, float* gates, void* stream);
 /* Counting sort of the (token, choice) pairs by expert: group_off [n_experts + 1], src_row [n_tokens * top] (token of
  * each sorted row), dest [n_tokens, top] (sorted row of each pair, -1 for chosen >= n_experts: identity experts own no
  * rows). One launch, no host sync. */
 int b200_moe_dispatch(const int* chosen, int n_tokens, int top, int n_experts, int* group_off, int* src_row, int* dest,
                       void* stream);
+/* the same; row_weight [n_tokens * top] (may be NULL) receives every sorted row's weight */
+int b200_moe_dispatch_weighted(const int* chosen, const float* weight, int n_tokens, int top, int n_experts, int* group_off, int* src_row,
+                               int* dest, float* row_weight, void* stream);
+/* dst[i, :] = src[rows[i], :] * scale[i], rounded once (routers whose weight multiplies the expert's input) */
+int b200_gather_rows_scaled(const void* src, const int* rows, const float* scale, void* dst, int n_rows, int width, int dtype, void* stream);
 /* dst[i, :] = src[rows[i], :] (both of `dtype`, contiguous rows of `width`): the sorted rows of b200_moe_dispatch side by side,
  * so that a dense GEMM can read one expert's group */
 int b200_gather_rows(const void* src, const int* rows, void* dst, int n_rows, int width, int dtype, void* stream);
@@ -227,6 +240,31 @@ typedef struct b200_parallel_residual_args {
 } b200_parallel_residual_args;
 int b200_parallel_residual(const b200_parallel_residual_args* a, void* stream);
 
+/* Token embedding into `streams` equal residual streams: out[t, s, :] = table[ids[t], :] * scale + sinusoids of the position, entry 2i
+ * sin(pos[t] * pi * turns[i]), entry 2i + 1 the cosine of the same (turns: device doubles [(width + 1) / 2], angle per position over
+ * pi; NULL: no sinusoids). table of `dtype`, out fp32 [n_tokens, streams, width]. */
+int b200_embed_streams(const int* ids, const int* pos, const void* table, float scale, const double* turns, float* out, int streams,
+                       int n_tokens, int width, int dtype, void* stream);
+/* Residual streams with learned connections (x fp32 [*, streams, width]), one launch between two sublayers:
+ *   y[t,:] = y1[t,:] + gate2[t] * y2[t,:] + sum_k weight[t,k] * expert_out[dest[t,k],:]     (every addend may be NULL; gate2, weight
+ *                                                                                           NULL: one)
+ *   x[t,k,:] <- sum_s mix[s,k] x[t,s,:] + w_out[k] * y[t,:]     (all streams at once from the old ones; skipped when mix is NULL)
+ *   u[t,:] = sum_s w_in[s] x[t,s,:]                             (the new streams; w_in NULL: their sum)
+ *   sum_out[t,:] = u[t,:] (fp32, may be NULL);  out[t,:] = u / sqrt(mean(u^2) + eps) * w   (as out_dtype; skipped when w is NULL)
+ * With `rows` (mix NULL) the call only reads: out[i,:] from x[rows[i]]. mix fp32 [streams, streams] (from, to), w_out, w_in [streams];
+ * at most 16 streams and 16 experts per token. */
+typedef struct b200_hyper_residual_args {
+    float* x; int streams;
+    const float* mix; const float* w_out;
+    const float* y1; const float* y2; const float* gate2;
+    const float* expert_out; const int* dest; const float* weight; int top;
+    const float* w_in; const int* rows;
+    const float* w; float eps;
+    void* out; int out_dtype; float* sum_out;
+    int n_rows, width;
+} b200_hyper_residual_args;
+int b200_hyper_residual(const b200_hyper_residual_args* a, void* stream);
+
 /* Dense feed-forward activation of normed powers: out[t,:] = c[0] N(z) + c[1] N(z^2) + c[2] N(z^3) + c[3], z = z[t,:] (fp32
  * [n_rows, width]), powers element by element, N v = v / sqrt(mean(v^2) + eps) over the row; out of out_dtype. */
 int b200_poly_norm(const float* z, const float* c4, float eps, void* out, int n_rows, int width, int out_dtype, void* stream);
@@ -272,6 +310,11 @@ typedef struct b200_qk_prepare_args {
        vdim dimensions (pairs in v_rot_layout) before the store. Both may be NULL. */
     const float* bias;
     const float* v_cos; const float* v_sin; int v_rot_layout;
+    /* norm_rows != 0: q_norm [heads*dim] and k_norm [kv_heads*dim] are the weights of ONE RMS norm over the whole query and one over
+       the whole key projection (before the split into heads) instead of one per head; no convolution then, and k_pool may be NULL:
+       queries only, for layers that read another layer's keys.
+       temp_every > 0: the queries of position p are multiplied by 1 + temp_coef * ln(floor((p + 1) / temp_every) + 1). */
+    int norm_rows; float temp_coef; int temp_every;
 } b200_qk_prepare_args;
 int b200_qk_prepare(const b200_qk_prepare_args* a, void* stream);
 /* The last taps-1 inputs of every sequence of the step go to their ring places (end[t] = the sequence's length after
@@ -315,6 +358,10 @@ typedef struct b200_paged_attention_args {
        b200_mixed_attention_workspace_bytes sizes; single tokens, fp32 and calls without workspace run on a kernel whose CTA
        (or cluster of CTAs, sharing the context) holds all heads of a token. */
     const float* head_temp; const float* head_mix;
+    /* sink (fp32 [heads] or NULL): head h's softmax denominator also holds exp(sink[h]), a learned score without key and value (not
+       scaled, no bias; not with denom_bias). dist_bias (fp32 [heads, dist_n] or NULL): dist_bias[h, min(p - j, dist_n - 1)] is added
+       to the scaled (and capped) score of key j at position p. Not with sigmoid_weights or head_mix. */
+    const float* sink; const float* dist_bias; int dist_n;
 } b200_paged_attention_args;
 size_t b200_paged_attention_workspace_bytes(int n_tokens, int heads, int vdim);
 /* longest_seen: most keys a token sees before the window is applied (the longest sequence); window 0: none */
@@ -343,6 +390,9 @@ int b200_retention(const b200_retention_args* a, void* stream);
  * dimension ld_gate) */
 int b200_unit_rms_gate(const float* o, const float* gate, long long ld_gate, void* out, int n_tokens, int heads, int vdim,
                        float eps, int out_dtype, void* stream);
+/* the same times a weight (fp32 [heads * vdim] or NULL); sigmoid_gate != 0: the gate is sigmoid(z) instead of silu(z) */
+int b200_head_rms_gate(const float* o, const float* gate, long long ld_gate, const float* w, int sigmoid_gate, void* out, int n_tokens,
+                       int heads, int vdim, float eps, int out_dtype, void* stream);
 /* Differential combination of two attention maps: o = a[t,h,0,:] - lambda * a[t,h,1,:]; out[t,h,:] = o / sqrt(mean(o^2) + eps)
  * * out_scale, as out_dtype. a fp32 [n_tokens, heads, 2, vdim]. */
 int b200_diff_combine(const float* a, float lambda, float eps, float out_scale, void* out, int n_tokens, int heads, int vdim,
@@ -450,6 +500,29 @@ int b200_ssd_scan(const b200_ssd_scan_args* a, void* stream);
  * equal parts. y fp32 [n_tokens, n], z fp32 with leading dimension ld_z, w fp32 [n]; out of out_dtype. */
 int b200_gated_group_rms(const float* y, const float* z, long long ld_z, const float* w, void* out, int n_tokens, int n, int parts,
                          float eps, int out_dtype, void* stream);
+
+/* Matrix memory with exponential input gates and sigmoid forget gates (the mLSTM cell), stabilised by a running maximum. Per entry (a
+ * run of consecutive tokens of one sequence) and head, with q = q_scale * proj[t, q_off + h * dim + :], k, v likewise (v at v_off + h *
+ * vdim), i = cap tanh((proj[t, i_off + h] + i_bias[h]) / cap) and f = log sigmoid(cap tanh((proj[t, f_off + h] + f_bias[h]) / cap)):
+ *   m' = max(f + m, i);  S <- exp(f + m - m') S + exp(i - m') k v^T;  n <- exp(f + m - m') n + exp(i - m') k
+ *   out[t, h, :] = S^T q / (max(|n . q|, exp(-m')) + 1e-6)
+ * state fp32 [n_slots, heads, dim, vdim] holds S, norm fp32 [n_slots, heads, b200_mlstm_norm_floats(dim, vdim)] holds n and m (its
+ * layout is the kernels' own); S, n and m start from zero when the entry starts at position 0 and stay in place for the next step.
+ * proj fp32 [n_tokens, ld_proj], out fp32 [n_tokens, heads * vdim].
+ * Entries walk token by token in fp32; with chunked != 0, a workspace and an entry of 128 tokens or more, the step takes the chunk
+ * form (64-token chunks on tf32 tensor-core products with fp32 accumulation; gates, maxima, states and everything between chunks
+ * stay fp32, the sums of the log gates are kept in double; dim at most 256). */
+typedef struct b200_mlstm_args {
+    const float* proj; long long ld_proj; int q_off, k_off, v_off, i_off, f_off;
+    const float* i_bias; const float* f_bias; float gate_cap, q_scale;
+    float* state; float* norm; float* out;
+    const int* ent_row; const int* ent_len; const int* slot; const int* pos;
+    int n_entries, n_tokens, heads, dim, vdim, longest_entry, chunked;
+    void* workspace; size_t workspace_bytes;
+} b200_mlstm_args;
+size_t b200_mlstm_norm_floats(int dim, int vdim);
+size_t b200_mlstm_workspace_bytes(int n_tokens, int n_entries, int heads, int dim, int vdim);
+int b200_mlstm(const b200_mlstm_args* a, void* stream);
 
 /* ---------------------------------------------------------------------------------------------
  * models

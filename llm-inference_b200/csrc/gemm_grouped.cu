@@ -4,7 +4,8 @@
 //                            (a head's slice of a wider activation is addressed in place, no copies)
 //   * groups               : blockIdx.z = group g owns rows [group_off[g], group_off[g+1]) of A and C and weight g
 //                            (the experts of a routed layer; the offsets live on the DEVICE, no host sync)
-//   * row gather           : A row r is a_rows[r] of the source (tokens sorted by expert are never materialised)
+//   * row gather           : A row r is a_rows[r] of the source (tokens sorted by expert are never materialised), times
+//                            row_scale[r] where given (routers whose weight multiplies an expert's input)
 //   * epilogues            : none | acc * sigmoid(aux) (output gate) | silu(acc_gate) * acc_up (GLU: the W tile holds
 //                            gate rows [0, N) and up rows [N, 2N) of the same features, the [M, 2N] intermediate is
 //                            never stored)
@@ -27,12 +28,18 @@ struct GG {
     long long lda, ldw, ldc, ld_aux, sA, sW, sC, s_aux;
     int M, N, K, epi;
     float epi_param;
+    const float* row_scale;
 };
 
 constexpr int GBM = 64, GBN = 64, GBK = 16;
 
 template <typename TC>
 __device__ __forceinline__ void gg_store(const GG& g, TC* C, long long row, int col, float v, float v2, long long aux_off) {
+    if (g.row_scale) {   // the row of A was meant to be scaled: the products are linear in it
+        const float f = g.row_scale[row];
+        v *= f;
+        v2 *= f;
+    }
     if (g.epi == B200_GG_SIGMOID_MUL) v *= 1.f / (1.f + expf(-g.aux[aux_off + row * g.ld_aux + col]));
     else if (g.epi == B200_GG_GLU) v = v / (1.f + expf(-v)) * v2;
     else if (g.epi == B200_GG_GLU_GELU) v = gelu_tanh_f(v) * v2;
@@ -390,7 +397,7 @@ extern "C" int b200_gemm_grouped(const b200_gemm_grouped_args* p, void* stream) 
     g.A = p->A; g.W = p->W; g.C = p->C; g.aux = p->aux; g.a_rows = p->a_rows; g.group_off = p->group_off;
     g.lda = p->lda; g.ldw = p->ldw; g.ldc = p->ldc; g.ld_aux = p->ld_aux;
     g.sA = p->stride_a; g.sW = p->stride_w; g.sC = p->stride_c; g.s_aux = p->stride_aux;
-    g.M = p->M; g.N = p->N; g.K = p->K; g.epi = p->epi; g.epi_param = p->epi_param;
+    g.M = p->M; g.N = p->N; g.K = p->K; g.epi = p->epi; g.epi_param = p->epi_param; g.row_scale = p->row_scale;
     if (p->epi == B200_GG_GLU_CLAMP && !(p->epi_param > 0.f)) return B200_EINVAL;
     // groups: M is the largest number of rows one group can own (the grid covers it; CTAs beyond a group's rows leave)
     dim3 grid((p->N + GBN - 1) / GBN, (p->M + GBM - 1) / GBM, p->batch);

@@ -266,7 +266,8 @@ int StepRunner::expert_rows(const ExpertGroups& g, int k, std::string& err) {
         group_off_cap_ = g.experts + 1;
     }
     cudaMemcpyAsync(group_off_host_, g.group_off, (size_t)(g.experts + 1) * sizeof(int), cudaMemcpyDeviceToHost, lane(k));
-    const int rc = b200_gather_rows(g.h, g.src_row, g.gathered, g.rows * g.top, D_, dtype_, lane(k));
+    const int rc = g.row_scale ? b200_gather_rows_scaled(g.h, g.src_row, g.row_scale, g.gathered, g.rows * g.top, D_, dtype_, lane(k))
+                               : b200_gather_rows(g.h, g.src_row, g.gathered, g.rows * g.top, D_, dtype_, lane(k));
     if (rc != B200_OK) { err = "b200_gather_rows failed"; return rc; }
     const cudaError_t e = cudaEventRecord(groups_ready_, lane(k));
     if (e != cudaSuccess) { err = std::string("step: ") + cudaGetErrorString(e); return (int)e; }

@@ -175,6 +175,7 @@ protected:
         const int* group_off; const int* src_row;
         const void* w_up; const void* w_down;   // [experts, ff (GLU: 2 ff), D] and [experts, D, ff]
         void* gathered; void* act; float* out;
+        const float* row_scale = nullptr;   // per sorted row: the expert reads its input times this
     };
     bool experts_fit_streams(int rows, int ff, bool glu) const {
         return dtype_ == B200_BF16 && !capturing_ && rows >= 1024 && D_ % 8 == 0 && ff % (glu ? 128 : 8) == 0;

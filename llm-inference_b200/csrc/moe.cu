@@ -1,6 +1,7 @@
 // Mixture-of-experts plumbing around b200_gemm_grouped: routers (softmax over all outputs with a corrected choice and
-// identity experts; a choice on the biased logits with a softmax over the chosen ones; or softmax over all with the choice
-// limited to the best groups of experts and renormalised weights), counting sort of the (token, choice) pairs by expert, and the fp32 residual update that gathers every
+// identity experts; a choice on the biased logits with a softmax over the chosen ones; softmax over all with the choice
+// limited to the best groups of experts and renormalised weights; or sigmoids that are weights as they are, beside the gates of
+// shared experts), counting sort of the (token, choice) pairs by expert, and the fp32 residual update that gathers every
 // token's expert rows back in a fixed order (no atomics: a token's sum does not depend on the batch around it).
 #include "b200_serve.h"
 #include "common.cuh"
@@ -80,17 +81,18 @@ __global__ void __launch_bounds__(512) moe_route_kernel(const T* __restrict__ h,
                                                         const float* __restrict__ corr, const float* __restrict__ bias,
                                                         int on_logits, int width, int n_out, int top,
                                                         float scale, int groups, int keep, int* __restrict__ chosen,
-                                                        float* __restrict__ weight) {
+                                                        float* __restrict__ weight, int sigmoids = 0, int n_gates = 0, float* __restrict__ gates = nullptr) {
     extern __shared__ float z[];   // z[n_out] | pick[n_out] | x[width]
-    float* pick = z + n_out;
-    float* xs = pick + n_out;
+    const int n_all = n_out + n_gates;   // the rows of w_router behind the experts' are gates of their own
+    float* pick = z + n_all;
+    float* xs = pick + n_all;
     const int t = blockIdx.x, warp = threadIdx.x / 32, lane = threadIdx.x % 32;
     const T* x = h + (size_t)t * width;
     // the token's input once in shared memory as fp32, then four independent partial sums per lane
     for (int i = threadIdx.x; i < width; i += blockDim.x) xs[i] = DT<T>::to_f(x[i]);
     __syncthreads();
     const int nw = blockDim.x / 32;
-    for (int o = warp; o < n_out; o += nw) {
+    for (int o = warp; o < n_all; o += nw) {
         const float* w = wr + (size_t)o * width;
         float d0 = 0.f, d1 = 0.f, d2 = 0.f, d3 = 0.f;
         int i = lane;
@@ -116,6 +118,22 @@ __global__ void __launch_bounds__(512) moe_route_kernel(const T* __restrict__ h,
     __syncthreads();
     if (groups > 0) {   // one warp: softmax, the best groups, the best experts inside them, renormalised weights
         if (warp == 0) route_in_groups(z, pick, n_out, top, groups, keep, lane, chosen + (size_t)t * top, weight + (size_t)t * top);
+        return;
+    }
+    if (sigmoids) {   // one warp: the largest logits, their sigmoids as weights
+        if (warp == 0) {
+            for (int k = lane; k < n_gates; k += 32) gates[(size_t)t * n_gates + k] = 1.f / (1.f + expf(-z[n_out + k]));
+            for (int k = 0; k < top; ++k) {
+                const int e = warp_argmax(z, n_out, lane);
+                __syncwarp();
+                if (lane == 0) {
+                    chosen[(size_t)t * top + k] = e;
+                    weight[(size_t)t * top + k] = 1.f / (1.f + expf(-z[e]));
+                    z[e] = -INFINITY;
+                }
+                __syncwarp();
+            }
+        }
         return;
     }
     if (threadIdx.x == 0 && on_logits) {   // the `top` largest logits, then a softmax over those alone
@@ -154,7 +172,8 @@ __global__ void __launch_bounds__(512) moe_route_kernel(const T* __restrict__ h,
 // computed independently of its neighbours, so the order does not reach the output.
 __global__ void __launch_bounds__(1024) moe_dispatch_kernel(const int* __restrict__ chosen, int n_pairs, int n_experts,
                                                             int top, int* __restrict__ group_off, int* __restrict__ src_row,
-                                                            int* __restrict__ dest) {
+                                                            int* __restrict__ dest, const float* __restrict__ weight,
+                                                            float* __restrict__ row_weight) {
     extern __shared__ int cnt[];   // count[n_experts] | cursor[n_experts]
     int* cursor = cnt + n_experts;
     for (int e = threadIdx.x; e < n_experts; e += blockDim.x) cnt[e] = 0;
@@ -180,6 +199,7 @@ __global__ void __launch_bounds__(1024) moe_dispatch_kernel(const int* __restric
         if (e < n_experts) {
             d = atomicAdd(&cursor[e], 1);
             src_row[d] = i / top;
+            if (row_weight) row_weight[d] = weight[i];
         }
         dest[i] = d;
     }
@@ -208,6 +228,27 @@ __global__ void __launch_bounds__(256) residual_combine_kernel(float* __restrict
     }
 }
 
+// dst[i, :] = src[rows[i], :] * scale[i] (fp32 product, rounded once)
+template <typename T>
+__global__ void __launch_bounds__(256) gather_rows_scaled_kernel(const T* __restrict__ src, const int* __restrict__ rows, const float* __restrict__ scale,
+                                                                T* __restrict__ dst, int width, int vec) {
+    constexpr int P = DT<T>::kPer16B;
+    const T* s = src + (size_t)rows[blockIdx.x] * width;
+    T* d = dst + (size_t)blockIdx.x * width;
+    const float f = scale[blockIdx.x];
+    if (vec) {
+        for (int i = threadIdx.x * P; i < width; i += blockDim.x * P) {
+            Pack16 pk = ld16(s + i);
+            T* e = reinterpret_cast<T*>(&pk);
+#pragma unroll
+            for (int k = 0; k < P; ++k) e[k] = DT<T>::from_f(DT<T>::to_f(e[k]) * f);
+            st16(d + i, pk);
+        }
+    } else {
+        for (int i = threadIdx.x; i < width; i += blockDim.x) d[i] = DT<T>::from_f(DT<T>::to_f(s[i]) * f);
+    }
+}
+
 // dst[i, :] = src[rows[i], :]: the rows of every expert's group side by side, so that a dense GEMM can read a group
 __global__ void __launch_bounds__(256) gather_rows_kernel(const unsigned char* __restrict__ src, const int* __restrict__ rows,
                                                          unsigned char* __restrict__ dst, size_t row_bytes, int vec) {
@@ -230,6 +271,38 @@ extern "C" int b200_gather_rows(const void* src, const int* rows, void* dst, int
     const size_t row_bytes = (size_t)width * (dtype == B200_BF16 ? 2 : 4);
     const int vec = row_bytes % 16 == 0 && (reinterpret_cast<uintptr_t>(src) & 15u) == 0 && (reinterpret_cast<uintptr_t>(dst) & 15u) == 0;
     gather_rows_kernel<<<n_rows, 256, 0, (cudaStream_t)stream>>>((const unsigned char*)src, rows, (unsigned char*)dst, row_bytes, vec);
+    count_launch();
+    return (int)cudaGetLastError();
+}
+
+extern "C" int b200_gather_rows_scaled(const void* src, const int* rows, const float* scale, void* dst, int n_rows, int width, int dtype, void* stream) {
+    if (!src || !rows || !scale || !dst || n_rows < 0 || width < 1 || (dtype != B200_BF16 && dtype != B200_F32)) return B200_EINVAL;
+    if (n_rows == 0) return B200_OK;
+    const int vec = ((size_t)width * (dtype == B200_BF16 ? 2 : 4)) % 16 == 0 && (reinterpret_cast<uintptr_t>(src) & 15u) == 0 && (reinterpret_cast<uintptr_t>(dst) & 15u) == 0;
+    cudaStream_t s = (cudaStream_t)stream;
+    if (dtype == B200_BF16) gather_rows_scaled_kernel<__nv_bfloat16><<<n_rows, 256, 0, s>>>((const __nv_bfloat16*)src, rows, scale, (__nv_bfloat16*)dst, width, vec);
+    else gather_rows_scaled_kernel<float><<<n_rows, 256, 0, s>>>((const float*)src, rows, scale, (float*)dst, width, vec);
+    count_launch();
+    return (int)cudaGetLastError();
+}
+
+extern "C" int b200_moe_route_sigmoid(const void* h, int h_dtype, const float* w_router, int n_tokens, int width, int n_out, int top, int n_gates,
+                                      int* chosen, float* weight, float* gates, void* stream) {
+    if (!h || !w_router || !chosen || !weight || n_tokens < 0 || width < 1 || n_out < 1 || top < 1 || top > n_out || n_gates < 0 || (n_gates && !gates))
+        return B200_EINVAL;
+    if (n_out + n_gates > 4096) return B200_EUNSUPPORTED;
+    if (n_tokens == 0) return B200_OK;
+    cudaStream_t s = (cudaStream_t)stream;
+    const size_t smem = ((size_t)2 * (n_out + n_gates) + width) * sizeof(float);
+    if (smem > 48 * 1024) return B200_EUNSUPPORTED;
+    if (h_dtype == B200_BF16)
+        moe_route_kernel<__nv_bfloat16><<<n_tokens, 512, smem, s>>>((const __nv_bfloat16*)h, w_router, nullptr, nullptr, 0, width, n_out, top, 1.f,
+                                                                   0, 0, chosen, weight, 1, n_gates, gates);
+    else if (h_dtype == B200_F32)
+        moe_route_kernel<float><<<n_tokens, 512, smem, s>>>((const float*)h, w_router, nullptr, nullptr, 0, width, n_out, top, 1.f, 0, 0, chosen,
+                                                           weight, 1, n_gates, gates);
+    else
+        return B200_EINVAL;
     count_launch();
     return (int)cudaGetLastError();
 }
@@ -298,10 +371,16 @@ extern "C" int b200_moe_route_groups(const void* h, int h_dtype, const float* w_
 
 extern "C" int b200_moe_dispatch(const int* chosen, int n_tokens, int top, int n_experts, int* group_off, int* src_row,
                                  int* dest, void* stream) {
+    return b200_moe_dispatch_weighted(chosen, nullptr, n_tokens, top, n_experts, group_off, src_row, dest, nullptr, stream);
+}
+
+extern "C" int b200_moe_dispatch_weighted(const int* chosen, const float* weight, int n_tokens, int top, int n_experts, int* group_off, int* src_row,
+                                          int* dest, float* row_weight, void* stream) {
+    if (row_weight && !weight) return B200_EINVAL;
     if (!chosen || !group_off || !src_row || !dest || n_tokens < 0 || top < 1 || n_experts < 0) return B200_EINVAL;
     if (n_experts > 4096) return B200_EUNSUPPORTED;
     moe_dispatch_kernel<<<1, 1024, (size_t)2 * (n_experts + 1) * sizeof(int), (cudaStream_t)stream>>>(
-        chosen, n_tokens * top, n_experts, top, group_off, src_row, dest);
+        chosen, n_tokens * top, n_experts, top, group_off, src_row, dest, weight, row_weight);
     count_launch();
     return (int)cudaGetLastError();
 }

@@ -18,6 +18,7 @@ struct PA {
     int chunk, maps, out_f32;
     int window, sigmoid; const float* head_bias;
     const float* head_temp; const float* head_mix;
+    const float* sink; const float* dist_bias; int dist_n;
 };
 // first key that position p sees
 __device__ __forceinline__ int pa_first_key(const PA& a, int p) {
@@ -26,6 +27,10 @@ __device__ __forceinline__ int pa_first_key(const PA& a, int p) {
 }
 // what the scores of head h are multiplied by
 __device__ __forceinline__ float pa_scale(const PA& a, int h) { return a.head_temp ? a.scale * a.head_temp[h] : a.scale; }
+// what the scaled score of a key `dist` positions back gains in head h
+__device__ __forceinline__ float pa_dist_bias(const PA& a, int h, int dist) {
+    return a.dist_bias ? a.dist_bias[(size_t)h * a.dist_n + min(dist, a.dist_n - 1)] : 0.f;
+}
 template <typename T>
 __device__ __forceinline__ void pa_store(const PA& a, size_t idx, float v) {
     if (a.out_f32) reinterpret_cast<float*>(a.out)[idx] = v;
@@ -59,7 +64,8 @@ __device__ __forceinline__ uint32_t pa_pack(float lo, float hi) {
     return *reinterpret_cast<const uint32_t*>(&h);
 }
 
-
+// tensor-core tiles with a distance bias and / or a learned sink (biased_attention.cu); -1: no tile for these sizes
+int biased_tile(const PA& a, cudaStream_t s);
 // b200_paged_attention with weights mixed across heads (mixed_attention.cu); a.head_mix is set
 int mixed_attention(const PA& a, int dtype, int longest_entry, int longest_context, void* workspace, size_t workspace_bytes, cudaStream_t s);
 

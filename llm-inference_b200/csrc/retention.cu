@@ -1,4 +1,5 @@
-// Retention (linear attention with a fixed decay per head and a carried state, no softmax) and the unit-RMS output gate.
+// Retention (linear attention with a fixed decay per head and a carried state, no softmax) and the unit-RMS output gate (which
+// can carry a weight and a sigmoid instead of the silu).
 // Everything here is fp32: the rotated q and k, the state, the decays and the sums.
 //
 //   retention_walk_kernel   one CTA per (entry, head, group of value columns): a thread owns one column of the state
@@ -284,10 +285,10 @@ __global__ void __launch_bounds__(256) retention_chunk_out_kernel(const RC rc) {
         }
 }
 
-// one warp per (token, head)
-template <typename T>
-__global__ void unit_rms_gate_kernel(const float* __restrict__ o, const float* __restrict__ gate, long long ld_gate, T* __restrict__ out,
-                                     int units, int heads, int vdim, float eps) {
+// one warp per (token, head); w [heads, vdim] may be NULL; the gate is silu(z) or (SIG) sigmoid(z)
+template <typename T, bool SIG>
+__global__ void unit_rms_gate_kernel(const float* __restrict__ o, const float* __restrict__ gate, long long ld_gate, const float* __restrict__ w,
+                                     T* __restrict__ out, int units, int heads, int vdim, float eps) {
     const int u = blockIdx.x * (blockDim.x / 32) + threadIdx.x / 32, lane = threadIdx.x % 32;
     if (u >= units) return;
     const int t = u / heads, h = u % heads;
@@ -300,8 +301,65 @@ __global__ void unit_rms_gate_kernel(const float* __restrict__ o, const float* _
     const float* g = gate + (size_t)t * ld_gate + (size_t)h * vdim;
     for (int i = lane; i < vdim; i += 32) {
         const float z = g[i];
-        out[(size_t)u * vdim + i] = DT<T>::from_f(src[i] * rinv * (z / (1.f + expf(-z))));
+        const float v = w ? src[i] * rinv * w[(size_t)h * vdim + i] : src[i] * rinv;
+        out[(size_t)u * vdim + i] = DT<T>::from_f(v * ((SIG ? 1.f : z) / (1.f + expf(-z))));
     }
+}
+
+// the same for heads in whole groups of four columns, at most 4 * 32 * PER of them: loads in flight together, the head in registers
+template <typename T, bool SIG, int PER>
+__global__ void __launch_bounds__(128) unit_rms_gate_reg_kernel(const float* __restrict__ o, const float* __restrict__ gate, long long ld_gate,
+                                                                const float* __restrict__ w, T* __restrict__ out, int units, int heads, int vdim,
+                                                                float eps) {
+    const int u = blockIdx.x * 4 + threadIdx.x / 32, lane = threadIdx.x % 32, quads = vdim / 4;
+    if (u >= units) return;
+    const int t = u / heads, h = u % heads;
+    const float4* src = reinterpret_cast<const float4*>(o + (size_t)u * vdim);
+    const float4* g = reinterpret_cast<const float4*>(gate + (size_t)t * ld_gate + (size_t)h * vdim);
+    const float4* wp = reinterpret_cast<const float4*>(w + (size_t)h * vdim);
+    float4 v[PER], z[PER], wv[PER];
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < PER; ++k) {
+        const int c = lane + 32 * k;
+        v[k] = z[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+        wv[k] = make_float4(1.f, 1.f, 1.f, 1.f);
+        if (c < quads) {
+            v[k] = src[c];
+            z[k] = g[c];
+            if (w) wv[k] = wp[c];
+        }
+        ss += v[k].x * v[k].x + v[k].y * v[k].y + v[k].z * v[k].z + v[k].w * v[k].w;
+    }
+#pragma unroll
+    for (int d = 16; d > 0; d >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, d);
+    const float rinv = 1.0f / sqrtf(ss / (float)vdim + eps);
+    T* dst = out + (size_t)u * vdim;
+#pragma unroll
+    for (int k = 0; k < PER; ++k) {
+        const int c = lane + 32 * k;
+        if (c >= quads) continue;
+        const float f[4] = {v[k].x * rinv * wv[k].x * ((SIG ? 1.f : z[k].x) / (1.f + expf(-z[k].x))), v[k].y * rinv * wv[k].y * ((SIG ? 1.f : z[k].y) / (1.f + expf(-z[k].y))),
+                            v[k].z * rinv * wv[k].z * ((SIG ? 1.f : z[k].z) / (1.f + expf(-z[k].z))), v[k].w * rinv * wv[k].w * ((SIG ? 1.f : z[k].w) / (1.f + expf(-z[k].w)))};
+        if constexpr (sizeof(T) == 4) reinterpret_cast<float4*>(dst)[c] = make_float4(f[0], f[1], f[2], f[3]);
+        else {
+            const __nv_bfloat162 lo = __floats2bfloat162_rn(f[0], f[1]), hi = __floats2bfloat162_rn(f[2], f[3]);
+            reinterpret_cast<uint2*>(dst)[c] = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+        }
+    }
+}
+
+template <typename T, bool SIG>
+static void launch_unit_rms(const float* o, const float* gate, long long ld_gate, const float* w, T* out, int units, int heads, int vdim, float eps,
+                            cudaStream_t s) {
+    auto al16 = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15u) == 0; };
+    const unsigned grid = (unsigned)((units + 3) / 4);
+    if (vdim % 4 == 0 && vdim <= 512 && ld_gate % 4 == 0 && al16(o) && al16(gate) && al16(w) && al16(out)) {
+        if (vdim <= 128) unit_rms_gate_reg_kernel<T, SIG, 1><<<grid, 128, 0, s>>>(o, gate, ld_gate, w, out, units, heads, vdim, eps);
+        else if (vdim <= 256) unit_rms_gate_reg_kernel<T, SIG, 2><<<grid, 128, 0, s>>>(o, gate, ld_gate, w, out, units, heads, vdim, eps);
+        else unit_rms_gate_reg_kernel<T, SIG, 4><<<grid, 128, 0, s>>>(o, gate, ld_gate, w, out, units, heads, vdim, eps);
+    } else
+        unit_rms_gate_kernel<T, SIG><<<grid, 128, 0, s>>>(o, gate, ld_gate, w, out, units, heads, vdim, eps);
 }
 
 }  // namespace b200
@@ -364,14 +422,24 @@ extern "C" int b200_retention(const b200_retention_args* p, void* stream) {
 
 extern "C" int b200_unit_rms_gate(const float* o, const float* gate, long long ld_gate, void* out, int n_tokens, int heads, int vdim,
                                   float eps, int out_dtype, void* stream) {
+    return b200_head_rms_gate(o, gate, ld_gate, nullptr, 0, out, n_tokens, heads, vdim, eps, out_dtype, stream);
+}
+
+extern "C" int b200_head_rms_gate(const float* o, const float* gate, long long ld_gate, const float* w, int sigmoid_gate, void* out, int n_tokens,
+                                  int heads, int vdim, float eps, int out_dtype, void* stream) {
     if (!o || !gate || !out || n_tokens < 0 || heads < 1 || vdim < 1) return B200_EINVAL;
+    if (out_dtype != B200_BF16 && out_dtype != B200_F32) return B200_EINVAL;
     if (n_tokens == 0) return B200_OK;
     const int units = n_tokens * heads;
-    const dim3 grid((units + 3) / 4);
     cudaStream_t s = (cudaStream_t)stream;
-    if (out_dtype == B200_BF16) unit_rms_gate_kernel<__nv_bfloat16><<<grid, 128, 0, s>>>(o, gate, ld_gate, (__nv_bfloat16*)out, units, heads, vdim, eps);
-    else if (out_dtype == B200_F32) unit_rms_gate_kernel<float><<<grid, 128, 0, s>>>(o, gate, ld_gate, (float*)out, units, heads, vdim, eps);
-    else return B200_EINVAL;
+    using bf = __nv_bfloat16;
+    if (out_dtype == B200_BF16) {
+        if (sigmoid_gate) launch_unit_rms<bf, true>(o, gate, ld_gate, w, (bf*)out, units, heads, vdim, eps, s);
+        else launch_unit_rms<bf, false>(o, gate, ld_gate, w, (bf*)out, units, heads, vdim, eps, s);
+    } else {
+        if (sigmoid_gate) launch_unit_rms<float, true>(o, gate, ld_gate, w, (float*)out, units, heads, vdim, eps, s);
+        else launch_unit_rms<float, false>(o, gate, ld_gate, w, (float*)out, units, heads, vdim, eps, s);
+    }
     count_launch();
     return (int)cudaGetLastError();
 }

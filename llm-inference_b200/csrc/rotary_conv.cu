@@ -35,7 +35,13 @@ struct QkPrep {
     int v_heads, vdim; long long v_off;
     const float* bias; const float* v_cos; const float* v_sin; int v_layout;
     int vals_per_warp;   // floats of shared memory per warp: max(dim, vdim)
+    float temp_coef; int temp_every;
 };
+
+// what the queries of position p are multiplied by
+__device__ __forceinline__ float query_temp(const QkPrep& a, int p) {
+    return a.temp_every > 0 ? 1.f + a.temp_coef * logf((float)((p + 1) / a.temp_every + 1)) : 1.f;
+}
 
 // One warp per (token, head unit): units [0, heads) are query heads, [heads, heads + kv_heads) key heads; a lane owns the
 // dimensions lane, lane + 32, ... (coalesced loads and stores); the head's sum of squares is a warp reduction and the
@@ -152,8 +158,97 @@ __global__ void __launch_bounds__(kPrepWarps * 32) qk_prepare_kernel(const QkPre
     __syncwarp();
     const int nf = a.rot_dims / 2;
     T* dst = is_k ? reinterpret_cast<T*>(a.k_pool) + cache_row * dim : reinterpret_cast<T*>(a.q_out) + ((size_t)t * a.heads + u) * dim;
+    const float mul = is_k ? 1.f : query_temp(a, p);
     for (int i = lane; i < dim; i += 32)
-        dst[i] = DT<T>::from_f(rotary_component(vals, i, a.rot_dims, a.rot_layout, a.cos + (size_t)t * nf, a.sin + (size_t)t * nf));
+        dst[i] = DT<T>::from_f(rotary_component(vals, i, a.rot_dims, a.rot_layout, a.cos + (size_t)t * nf, a.sin + (size_t)t * nf) * mul);
+}
+
+// Norms over the WHOLE query and the whole key projection (before they are split into heads): one CTA per token sums the squares of
+// both parts, then norms, turns (through shared memory, where the design rotates), scales the queries and scatters q, k and the
+// projected values. VEC consecutive dimensions per thread and step.
+constexpr int kRowPrepThreads = 256;
+template <typename T, int VEC>
+__device__ __forceinline__ void prep_store(T* dst, const float (&v)[VEC]) {
+    if constexpr (VEC == 1) dst[0] = DT<T>::from_f(v[0]);
+    else if constexpr (sizeof(T) == 4) *reinterpret_cast<float4*>(dst) = make_float4(v[0], v[1], v[2], v[3]);
+    else {
+        const __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1]), hi = __floats2bfloat162_rn(v[2], v[3]);
+        *reinterpret_cast<uint2*>(dst) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+    }
+}
+template <int VEC>
+__device__ __forceinline__ void prep_load(float (&v)[VEC], const float* src) {
+    if constexpr (VEC == 1) v[0] = src[0];
+    else {
+        const float4 f = *reinterpret_cast<const float4*>(src);
+        v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
+    }
+}
+template <typename T, int VEC>
+__global__ void __launch_bounds__(kRowPrepThreads) qk_row_prepare_kernel(const QkPrep a) {
+    extern __shared__ __align__(16) float prep_sm[];   // rotated designs: the normed q and k of the token
+    __shared__ float red[2][kRowPrepThreads / 32];
+    const int t = blockIdx.x, dim = a.dim, nq = a.heads * dim, nk = a.kv_heads * dim, nv = a.v_heads * a.vdim, p = a.pos[t];
+    const float* row = a.proj + (size_t)t * a.ld_proj;
+    float sq = 0.f, sk = 0.f;
+    for (int i = threadIdx.x * VEC; i < nq + nk; i += kRowPrepThreads * VEC) {
+        float v[VEC];
+        prep_load<VEC>(v, row + i);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+            if (a.bias) v[e] += a.bias[i + e];
+            if (i < nq) sq += v[e] * v[e];
+            else sk += v[e] * v[e];
+        }
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+        sq += __shfl_xor_sync(0xffffffffu, sq, o);
+        sk += __shfl_xor_sync(0xffffffffu, sk, o);
+    }
+    if (threadIdx.x % 32 == 0) { red[0][threadIdx.x / 32] = sq; red[1][threadIdx.x / 32] = sk; }
+    __syncthreads();
+    sq = sk = 0.f;
+    for (int w = 0; w < kRowPrepThreads / 32; ++w) { sq += red[0][w]; sk += red[1][w]; }
+    const float rq = a.q_norm ? 1.0f / sqrtf(sq / (float)nq + a.eps) : 1.f, rk = a.k_norm && nk > 0 ? 1.0f / sqrtf(sk / (float)nk + a.eps) : 1.f;
+    const float mul = query_temp(a, p);
+    size_t cache_row = 0;
+    if (nk + nv > 0) cache_row = (size_t)a.pages[(size_t)a.slot[t] * a.max_pages + p / a.page_rows] * a.page_rows + p % a.page_rows;
+    T* qd = reinterpret_cast<T*>(a.q_out) + (size_t)t * nq;
+    T* kd = reinterpret_cast<T*>(a.k_pool) + cache_row * nk;
+    for (int i = threadIdx.x * VEC; i < nq + nk; i += kRowPrepThreads * VEC) {
+        const bool is_k = i >= nq;
+        const float* nw = is_k ? a.k_norm : a.q_norm;
+        const int c = is_k ? i - nq : i;
+        float v[VEC];
+        prep_load<VEC>(v, row + i);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+            if (a.bias) v[e] += a.bias[i + e];
+            v[e] *= is_k ? rk : rq;
+            if (nw) v[e] *= nw[c + e];
+            if (a.rot_dims) prep_sm[i + e] = v[e];
+            else if (!is_k) v[e] *= mul;
+        }
+        if (!a.rot_dims) prep_store<T, VEC>(is_k ? kd + c : qd + c, v);
+    }
+    for (int i = threadIdx.x * VEC; i < nv; i += kRowPrepThreads * VEC) {
+        float v[VEC];
+        prep_load<VEC>(v, row + a.v_off + i);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e)
+            if (a.bias) v[e] += a.bias[a.v_off + i + e];
+        prep_store<T, VEC>(reinterpret_cast<T*>(a.v_pool) + cache_row * nv + i, v);
+    }
+    if (!a.rot_dims) return;
+    __syncthreads();
+    const int nf = a.rot_dims / 2;
+    for (int i = threadIdx.x; i < nq + nk; i += kRowPrepThreads) {
+        const bool is_k = i >= nq;
+        const float v = rotary_component(prep_sm + i / dim * dim, i % dim, a.rot_dims, a.rot_layout, a.cos + (size_t)t * nf, a.sin + (size_t)t * nf);
+        if (is_k) kd[i - nq] = DT<T>::from_f(v);
+        else qd[i] = DT<T>::from_f(v * mul);
+    }
 }
 
 // Without convolution and head norm the preparation is a rotation and three scatters: a thread per four consecutive
@@ -240,7 +335,7 @@ extern "C" int b200_rope_angles(const int* pos, int n_tokens, const double* freq
 }
 
 extern "C" int b200_qk_prepare(const b200_qk_prepare_args* p, void* stream) {
-    if (!p || !p->proj || !p->q_out || !p->k_pool || !p->pages || !p->slot || !p->pos || p->n_tokens < 0 || p->heads < 1 ||
+    if (!p || !p->proj || !p->q_out || (!p->k_pool && (!p->norm_rows || p->v_heads)) || !p->pages || !p->slot || !p->pos || p->n_tokens < 0 || p->heads < 1 ||
         p->kv_heads < 1 || p->dim < 1 || p->page_rows < 1)
         return B200_EINVAL;
     if (p->conv_w && (p->taps < 1 || !p->start || (p->taps > 1 && !p->conv_state))) return B200_EINVAL;
@@ -248,6 +343,8 @@ extern "C" int b200_qk_prepare(const b200_qk_prepare_args* p, void* stream) {
     if (p->v_heads < 0 || (p->v_heads > 0 && (!p->v_pool || p->vdim < 1 || p->v_from_conv || p->v_off < 0))) return B200_EINVAL;
     if (p->rot_dims < 0 || (p->rot_dims & 1) || p->rot_dims > p->dim || (p->rot_dims && (!p->cos || !p->sin))) return B200_EINVAL;
     if (p->rot_layout != B200_ROPE_HALF && p->rot_layout != B200_ROPE_INTERLEAVED) return B200_EINVAL;
+    if (p->norm_rows && (p->conv_w || p->v_from_conv || p->v_cos)) return B200_EINVAL;
+    if (p->temp_every < 0) return B200_EINVAL;
     if (p->bias && p->conv_w) return B200_EINVAL;   // carried convolution inputs are raw projections
     if ((p->v_cos || p->v_sin) && (!p->v_cos || !p->v_sin || p->v_heads < 1 ||
                                    (p->v_rot_layout != B200_ROPE_HALF && p->v_rot_layout != B200_ROPE_INTERLEAVED)))
@@ -256,12 +353,29 @@ extern "C" int b200_qk_prepare(const b200_qk_prepare_args* p, void* stream) {
     QkPrep a{p->proj, p->ld_proj, p->conv_w, p->taps, p->conv_state, p->q_norm, p->k_norm, p->eps, p->cos, p->sin, p->rot_dims,
              p->rot_layout, p->q_out, p->k_pool, p->v_pool, p->v_from_conv, p->update_state_inline ? const_cast<float*>(p->conv_state) : nullptr, p->pages, p->max_pages, p->page_rows, p->slot, p->pos,
              p->start, p->heads, p->kv_heads, p->dim, p->v_heads, p->vdim, p->v_off, p->bias, p->v_cos, p->v_sin, p->v_rot_layout,
-             p->v_heads > 0 && p->vdim > p->dim ? p->vdim : p->dim};
+             p->v_heads > 0 && p->vdim > p->dim ? p->vdim : p->dim, p->temp_coef, p->temp_every};
     if (a.conv_w && a.taps == 1) a.conv_state = a.proj;   // never read: every input of a one-tap filter is the token's own
     cudaStream_t s = (cudaStream_t)stream;
+    auto al16 = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15u) == 0; };
+    if (p->norm_rows) {
+        if (!p->k_pool) a.kv_heads = 0;
+        const size_t smem = p->rot_dims ? (size_t)(a.heads + a.kv_heads) * p->dim * sizeof(float) : 0;
+        if (smem > 48 * 1024 - 128) return B200_EUNSUPPORTED;
+        const bool vec = p->dim % 4 == 0 && p->ld_proj % 4 == 0 && al16(p->proj) && al16(p->q_out) && al16(p->k_pool) &&
+                         (p->v_heads == 0 || (p->vdim % 4 == 0 && p->v_off % 4 == 0 && al16(p->v_pool)));
+        if (p->dtype == B200_BF16) {
+            if (vec) qk_row_prepare_kernel<__nv_bfloat16, 4><<<p->n_tokens, kRowPrepThreads, smem, s>>>(a);
+            else qk_row_prepare_kernel<__nv_bfloat16, 1><<<p->n_tokens, kRowPrepThreads, smem, s>>>(a);
+        } else if (p->dtype == B200_F32) {
+            if (vec) qk_row_prepare_kernel<float, 4><<<p->n_tokens, kRowPrepThreads, smem, s>>>(a);
+            else qk_row_prepare_kernel<float, 1><<<p->n_tokens, kRowPrepThreads, smem, s>>>(a);
+        } else
+            return B200_EINVAL;
+        count_launch();
+        return (int)cudaGetLastError();
+    }
     {   // rotation and scatters only, everything in whole groups of four: the vector kernel
-        auto al16 = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15u) == 0; };
-        const bool plain = !p->conv_w && !p->q_norm && !p->k_norm && !p->bias && !p->v_cos && p->rot_layout == B200_ROPE_HALF && p->dim % 4 == 0 && p->rot_dims % 8 == 0 &&
+        const bool plain = !p->temp_every && !p->conv_w && !p->q_norm && !p->k_norm && !p->bias && !p->v_cos && p->rot_layout == B200_ROPE_HALF && p->dim % 4 == 0 && p->rot_dims % 8 == 0 &&
                            p->ld_proj % 4 == 0 && al16(p->proj) && al16(p->q_out) && al16(p->k_pool) &&
                            (p->v_heads == 0 || (p->vdim % 4 == 0 && p->v_off % 4 == 0 && al16(p->v_pool))) &&
                            (p->dtype == B200_BF16 || p->dtype == B200_F32);

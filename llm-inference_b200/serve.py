@@ -19,7 +19,7 @@ class GemmGroupedArgs(C.Structure):
                 ("lda", _ll), ("ldw", _ll), ("ldc", _ll), ("ld_aux", _ll),
                 ("stride_a", _ll), ("stride_w", _ll), ("stride_c", _ll), ("stride_aux", _ll),
                 ("M", _i), ("N", _i), ("K", _i), ("batch", _i), ("trans_b", _i), ("epi", _i),
-                ("a_dtype", _i), ("w_dtype", _i), ("c_dtype", _i), ("epi_param", _f)]
+                ("a_dtype", _i), ("w_dtype", _i), ("c_dtype", _i), ("epi_param", _f), ("row_scale", _vp)]
 
 
 class QkPrepareArgs(C.Structure):
@@ -30,7 +30,8 @@ class QkPrepareArgs(C.Structure):
                 ("pages", _vp), ("max_pages", _i), ("page_rows", _i), ("slot", _vp), ("pos", _vp), ("start", _vp),
                 ("n_tokens", _i), ("heads", _i), ("kv_heads", _i), ("dim", _i), ("dtype", _i), ("update_state_inline", _i),
                 ("v_heads", _i), ("vdim", _i), ("v_off", _ll),
-                ("bias", _vp), ("v_cos", _vp), ("v_sin", _vp), ("v_rot_layout", _i)]
+                ("bias", _vp), ("v_cos", _vp), ("v_sin", _vp), ("v_rot_layout", _i),
+                ("norm_rows", _i), ("temp_coef", _f), ("temp_every", _i)]
 
 
 class PagedAttentionArgs(C.Structure):
@@ -40,7 +41,8 @@ class PagedAttentionArgs(C.Structure):
                 ("scale", _f), ("softcap", _f), ("denom_bias", _f), ("dtype", _i), ("longest_entry", _i),
                 ("longest_context", _i), ("workspace", _vp), ("workspace_bytes", _sz),
                 ("chunk", _i), ("maps", _i), ("out_f32", _i),
-                ("window", _i), ("sigmoid_weights", _i), ("head_bias", _vp), ("head_temp", _vp), ("head_mix", _vp)]
+                ("window", _i), ("sigmoid_weights", _i), ("head_bias", _vp), ("head_temp", _vp), ("head_mix", _vp),
+                ("sink", _vp), ("dist_bias", _vp), ("dist_n", _i)]
 
 
 class RmsnormResidualArgs(C.Structure):
@@ -114,6 +116,22 @@ class SsdScanArgs(C.Structure):
                 ("chunked", _i), ("workspace", _vp), ("workspace_bytes", _sz)]
 
 
+class HyperResidualArgs(C.Structure):
+    """mirror of ``b200_hyper_residual_args``"""
+    _fields_ = [("x", _vp), ("streams", _i), ("mix", _vp), ("w_out", _vp), ("y1", _vp), ("y2", _vp), ("gate2", _vp),
+                ("expert_out", _vp), ("dest", _vp), ("weight", _vp), ("top", _i), ("w_in", _vp), ("rows", _vp), ("w", _vp), ("eps", _f),
+                ("out", _vp), ("out_dtype", _i), ("sum_out", _vp), ("n_rows", _i), ("width", _i)]
+
+
+class MlstmArgs(C.Structure):
+    """mirror of ``b200_mlstm_args``"""
+    _fields_ = [("proj", _vp), ("ld_proj", _ll), ("q_off", _i), ("k_off", _i), ("v_off", _i), ("i_off", _i), ("f_off", _i),
+                ("i_bias", _vp), ("f_bias", _vp), ("gate_cap", _f), ("q_scale", _f), ("state", _vp), ("norm", _vp), ("out", _vp),
+                ("ent_row", _vp), ("ent_len", _vp), ("slot", _vp), ("pos", _vp),
+                ("n_entries", _i), ("n_tokens", _i), ("heads", _i), ("dim", _i), ("vdim", _i), ("longest_entry", _i), ("chunked", _i),
+                ("workspace", _vp), ("workspace_bytes", _sz)]
+
+
 class ModelOptions(C.Structure):
     """mirror of ``b200_model_options``"""
     _fields_ = [("dtype", _i), ("max_tokens", _i), ("max_slots", _i), ("max_step_tokens", _i)]
@@ -171,6 +189,15 @@ SERVE_PROTOTYPES = {
     "b200_ssd_scan_workspace_bytes": (_sz, [_i, _i, _i, _i, _i, _i]),
     "b200_ssd_scan": (_i, [C.POINTER(SsdScanArgs), _vp]),
     "b200_gated_group_rms": (_i, [_vp, _vp, _ll, _vp, _vp, _i, _i, _i, _f, _i, _vp]),
+    "b200_moe_route_sigmoid": (_i, [_vp, _i, _vp, _i, _i, _i, _i, _i, _vp, _vp, _vp, _vp]),
+    "b200_moe_dispatch_weighted": (_i, [_vp, _vp, _i, _i, _i, _vp, _vp, _vp, _vp, _vp]),
+    "b200_gather_rows_scaled": (_i, [_vp, _vp, _vp, _vp, _i, _i, _i, _vp]),
+    "b200_embed_streams": (_i, [_vp, _vp, _vp, _f, _vp, _vp, _i, _i, _i, _i, _vp]),
+    "b200_hyper_residual": (_i, [C.POINTER(HyperResidualArgs), _vp]),
+    "b200_head_rms_gate": (_i, [_vp, _vp, _ll, _vp, _i, _vp, _i, _i, _i, _f, _i, _vp]),
+    "b200_mlstm_norm_floats": (_sz, [_i, _i]),
+    "b200_mlstm_workspace_bytes": (_sz, [_i, _i, _i, _i, _i]),
+    "b200_mlstm": (_i, [C.POINTER(MlstmArgs), _vp]),
     "b200_serve_last_error": (C.c_char_p, []),
     "b200_model_families": (C.c_char_p, []),
     "b200_model_open": (_vp, [C.c_char_p, C.POINTER(ModelOptions)]),
