@@ -14,7 +14,8 @@ Workloads:
   nekodra, musilorn: not BASELINE.json configs: prefill and decode tokens/s of the Nekodra / Musilorn family
         (include/b200_serve.h, random weights, --size s|m) beside the LLaMA engine at equal size; a line of its own shape.
   tomalix: the same for the Tomalix family, beside the Musilorn family at equal size.
-  sakevik, filipel: the same for the Sakevik / Filipel family, beside the Tomalix family at equal size.
+  sakevik, filipel, mazotar: the same for the Sakevik / Filipel / Mazotar family, beside the Tomalix family at equal size
+        (mazotar: and beside the Musilorn family).
   cfg3: prefill, batch 4 x 2048 prompt tokens per GPU (metric prefill_tokens_per_s; a step = one prompt
         pass of the whole model: tcgen05 GEMMs + flash context attention; roofline = tensor).
 `value`  : tokens/s with everything resident in HBM, CUDA events on the engine's stream, max over ranks.
@@ -48,9 +49,9 @@ def parse():
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=128)
     ap.add_argument("--warmup", type=int, default=8)
-    ap.add_argument("--workload", default="cfg2", choices=["cfg2", "cfg3", "cfg4", "cfg5", "nekodra", "musilorn", "tomalix", "sakevik", "filipel"])
+    ap.add_argument("--workload", default="cfg2", choices=["cfg2", "cfg3", "cfg4", "cfg5", "nekodra", "musilorn", "tomalix", "sakevik", "filipel", "mazotar"])
     ap.add_argument("--size", default="m", choices=["s", "m"],
-                    help="nekodra / musilorn / tomalix / sakevik / filipel: model shape (llm-inference_b200/bench_families.py SIZES, MUSILORN_SIZES, TOMALIX_SIZES, SAKEVIK_SIZES, FILIPEL_SIZES)")
+                    help="nekodra / musilorn / tomalix / sakevik / filipel / mazotar: model shape (llm-inference_b200/bench_families.py SIZES, MUSILORN_SIZES, TOMALIX_SIZES, SAKEVIK_SIZES, FILIPEL_SIZES, MAZOTAR_SIZES)")
     ap.add_argument("--prompt", type=int, default=2048, help="nekodra: prompt tokens of the prefill measurement")
     ap.add_argument("--comm", default="p2p", choices=["p2p", "nccl"],
                     help="cfg5: fused one-shot NVLink allreduce (product) or ncclAllReduce + AddResidual (baseline)")
@@ -906,8 +907,8 @@ def extras_multi_gpu(pkg, args, rank, world, local_rank, peak):
 # the B200 arm
 # --------------------------------------------------------------------------------------------
 def bench_family(args):
-    """--workload nekodra | musilorn | tomalix | sakevik | filipel: prefill and decode tokens/s of that family (include/b200_serve.h) beside the LLaMA
-    engine (tomalix: beside the Musilorn family; sakevik, filipel: beside the Tomalix family) at equal size; one JSON line of its own shape (the default workload and its line stay as they are)."""
+    """--workload nekodra | musilorn | tomalix | sakevik | filipel | mazotar: prefill and decode tokens/s of that family (include/b200_serve.h) beside the LLaMA
+    engine (tomalix: beside the Musilorn family; sakevik, filipel, mazotar: beside the Tomalix family) at equal size; one JSON line of its own shape (the default workload and its line stay as they are)."""
     from __graft_entry__ import load_package
     pkg = load_package()
     from llm_inference_b200 import bench_families
@@ -919,7 +920,7 @@ def bench_family(args):
 
 def main():
     args = parse()
-    if args.workload in ("nekodra", "musilorn", "tomalix", "sakevik", "filipel"):
+    if args.workload in ("nekodra", "musilorn", "tomalix", "sakevik", "filipel", "mazotar"):
         return bench_family(args)
     wl = workload(args)
     rank = int(os.environ.get("RANK", "0"))

@@ -1,6 +1,6 @@
 """Prefill and decode throughput of a model family served through include/b200_serve.h, beside the LLaMA engine at
 equal size (same width, heads, layers, vocabulary and the same feed-forward width per token), random weights.
-Called by bench.py --workload nekodra | musilorn | tomalix | sakevik | filipel; prints one JSON line."""
+Called by bench.py --workload nekodra | musilorn | tomalix | sakevik | filipel | mazotar; prints one JSON line."""
 import json
 import os
 import tempfile
@@ -83,6 +83,22 @@ FILIPEL_SIZES = {
 }
 
 
+def mazotar_layers(width, heads, kv_heads, dim, ff, expert_ff, mem_heads, mem_dim, mem_vdim, **_):
+    """four layers: a matrix memory with a dense feed-forward; attention with 16 routed experts of which a token uses three, beside a
+    shared one of their size; attention with a dense feed-forward; attention on the second layer's keys with a dense one"""
+    att = dict(type="attention", heads=heads, kv_heads=kv_heads, dim=dim, vdim=dim)
+    return [dict(type="mlstm", heads=mem_heads, dim=mem_dim, vdim=mem_vdim, ff=ff), dict(att, ff=(expert_ff, 16, 3, expert_ff)),
+            dict(att, ff=ff), dict(att, kv_from=1, ff=ff)]
+
+
+# a gated unit holds three matrices where the squared-relu unit of Tomalix holds two: two thirds of its hidden width (rounded to 128);
+# three routed experts and the shared one stand against Tomalix's four
+MAZOTAR_SIZES = {
+    "s": dict(width=1024, heads=8, kv_heads=4, dim=128, ff=2688, expert_ff=640, mem_heads=4, mem_dim=128, mem_vdim=256, streams=4, n_layers=4, vocab=32000),
+    "m": dict(width=2048, heads=16, kv_heads=8, dim=128, ff=5504, expert_ff=1408, mem_heads=8, mem_dim=128, mem_vdim=256, streams=4, n_layers=4, vocab=32000),
+}
+
+
 def timed(fn, steps, warmup):
     import torch
     for _ in range(warmup):
@@ -106,6 +122,8 @@ def run(pkg, size="m", prompt=2048, batch=8, context=1024, steps=10, warmup=3, d
         return run_sakevik(pkg, size, prompt, batch, context, steps, warmup, dtype)
     if family == "filipel":
         return run_filipel(pkg, size, prompt, batch, context, steps, warmup, dtype)
+    if family == "mazotar":
+        return run_mazotar(pkg, size, prompt, batch, context, steps, warmup, dtype)
     sz = (MUSILORN_SIZES if family == "musilorn" else SIZES)[size]
     rng = np.random.default_rng(0)
     out = {"workload": family, "size": size, "shape": sz, "prompt": prompt, "decode_batch": batch, "decode_context": context,
@@ -265,4 +283,31 @@ def run_filipel(pkg, size, prompt, batch, context, steps, warmup, dtype):
         out["tomalix_equal_size"] = res
     except Exception as ex:   # the comparison must not take the family's own numbers down
         out["tomalix_equal_size"] = {"failed": f"{type(ex).__name__}: {ex}"}
+    return out
+
+
+def run_mazotar(pkg, size, prompt, batch, context, steps, warmup, dtype):
+    """The Mazotar family beside the closest existing one, Tomalix (the same serving layer and fp32 residual; grouped-query
+    attention, a recurrence with carried state, dense and routed feed-forwards), at equal width, heads, head size, layer count,
+    vocabulary and feed-forward weights per layer; and beside Musilorn at equal size, whose retention layer carries the same kind of
+    state (a matrix per head of the same sizes)."""
+    S = pkg.serve
+    sz = MAZOTAR_SIZES[size]
+    out = {"workload": "mazotar", "size": size, "shape": sz, "prompt": prompt, "decode_batch": batch, "decode_context": context,
+           "dtype": dtype, "data": "synthetic ids, random weights", "timing": "host clock around synchronous steps (each step ends "
+           "with the device-to-host copy of its results), after warm-up"}
+    cfg, w = S.random_mazotar(sz["width"], sz["vocab"], mazotar_layers(**sz), streams=sz["streams"])
+    out.update(serve_family(S, cfg, w, prompt, batch, context, steps, warmup, dtype, sz["vocab"]))
+    del w
+    tx, mu = dict(TOMALIX_SIZES[size]), dict(MUSILORN_SIZES[size])
+    for name, shape, make in (("tomalix", tx, lambda: S.random_tomalix(tx["width"], tx["vocab"], tomalix_layers(**tx))),
+                              ("musilorn", mu, lambda: S.random_musilorn(**mu))):
+        try:
+            cfg, w = make()
+            res = serve_family(S, cfg, w, prompt, batch, context, steps, warmup, dtype, shape["vocab"])
+            res["shape"] = shape
+            out[name + "_equal_size"] = res
+            del w
+        except Exception as ex:   # the comparison must not take the family's own numbers down
+            out[name + "_equal_size"] = {"failed": f"{type(ex).__name__}: {ex}"}
     return out

@@ -344,8 +344,8 @@ __global__ void __launch_bounds__(128) paged_attn_combine_kernel(const float* __
 
 // the (dim, vdim) pairs the tile kernel is built for: equal sizes, and values twice as wide as the keys
 static int launch_tile_for(const PA& a, cudaStream_t s) {
-    if (a.dim == a.vdim) return a.dim == 128 ? launch_tile<128, 128, false>(a, s) : a.dim == 64 ? launch_tile<64, 64, false>(a, s) : a.dim == 32 ? launch_tile<32, 32, false>(a, s) : -1;
-    if (a.vdim == 2 * a.dim) return a.dim == 128 ? launch_tile<128, 256, false>(a, s) : a.dim == 64 ? launch_tile<64, 128, false>(a, s) : a.dim == 32 ? launch_tile<32, 64, false>(a, s) : -1;
+    if (a.dim == a.vdim) return a.dim == 128 ? launch_tile<128, 128, kNoBias>(a, s) : a.dim == 64 ? launch_tile<64, 64, kNoBias>(a, s) : a.dim == 32 ? launch_tile<32, 32, kNoBias>(a, s) : -1;
+    if (a.vdim == 2 * a.dim) return a.dim == 128 ? launch_tile<128, 256, kNoBias>(a, s) : a.dim == 64 ? launch_tile<64, 128, kNoBias>(a, s) : a.dim == 32 ? launch_tile<32, 64, kNoBias>(a, s) : -1;
     return -1;
 }
 
@@ -378,7 +378,7 @@ extern "C" int b200_paged_attention(const b200_paged_attention_args* p, void* st
     if (smem > 48 * 1024) return B200_EUNSUPPORTED;
     auto al16 = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15u) == 0; };
     const char* env = getenv("B200_ATTN_ROWS");   // 1: every batch on the row kernel (debugging aid)
-    if (p->dtype == B200_BF16 && p->longest_entry != 1 && (p->sink || p->dist_bias) && p->dim % 8 == 0 && p->vdim % 8 == 0 && al16(p->q) && al16(p->out) &&
+    if (p->dtype == B200_BF16 && p->longest_entry != 1 && (p->sink || p->dist_bias) && !(p->softcap > 0.f) && p->dim % 8 == 0 && p->vdim % 8 == 0 && al16(p->q) && al16(p->out) &&
         al16(p->k_pool) && al16(p->v_pool) && !(env && env[0] == '1')) {
         const int rc = biased_tile(a, s);
         if (rc == 0) count_launch();

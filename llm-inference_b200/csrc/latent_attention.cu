@@ -297,6 +297,7 @@ __global__ void __launch_bounds__(256, NT <= 8 ? 2 : 1) latent_attn_tile_kernel(
                     dstbuf[kr * RS + c] = v;
                 }
             }
+            __syncwarp();   // the lanes close their group of copies together
             asm volatile("cp.async.commit_group;" ::: "memory");
         };
         // the rank is split between the warp groups 0-3 and 4-7 in the score phase (k steps of 16)

@@ -377,6 +377,7 @@ __global__ void __launch_bounds__(128) mixed_scores_kernel(const MxTile m) {
         const int r = i / CH, c = (i - r * CH) * 8;
         mx_cp16(Qs + r * RS + c, Q + ((size_t)(t0 + (r < rows ? r : 0)) * a.heads + h) * dim + (c < dim ? c : 0), r < rows && c < dim);
     }
+    __syncwarp();   // the lanes close their group of copies together
     asm volatile("cp.async.commit_group;" ::: "memory");
     __syncthreads();
     const bf* Kp = reinterpret_cast<const bf*>(a.k_pool);
@@ -412,6 +413,7 @@ __global__ void __launch_bounds__(128) mixed_scores_kernel(const MxTile m) {
                     const size_t row = ok ? (size_t)plist[j / a.page_rows] * a.page_rows + j % a.page_rows : 0;
                     mx_cp16(kd + kr * RS + c, Kp + (row * G + g) * dim + (ok ? c : 0), ok);
                 }
+            __syncwarp();   // the lanes close their group of copies together
             asm volatile("cp.async.commit_group;" ::: "memory");
         };
         __syncthreads();   // the buffers of the previous segment are no longer read
@@ -596,6 +598,7 @@ __global__ void __launch_bounds__(128) mixed_values_kernel(const MxTile m) {
                 const size_t row = !ok ? 0 : one_page ? base + kr : (size_t)plist[j / a.page_rows] * a.page_rows + j % a.page_rows;
                 mx_cp16(vd + kr * RSV + c, Vp + (row * G + g) * dv + (ok ? c : 0), ok);
             }
+            __syncwarp();   // the lanes close their group of copies together
             asm volatile("cp.async.commit_group;" ::: "memory");
         };
         __syncthreads();

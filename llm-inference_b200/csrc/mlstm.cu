@@ -228,6 +228,7 @@ __device__ __forceinline__ void ml_stage(float* dst, int stride, const float* sr
     }
 }
 __device__ __forceinline__ void ml_landed() {
+    __syncwarp();   // the lanes close their group of copies together
     asm volatile("cp.async.commit_group;\n\tcp.async.wait_group 0;" ::: "memory");
     __syncthreads();
 }

@@ -3,6 +3,8 @@
 // limited to the best groups of experts and renormalised weights; or sigmoids that are weights as they are, beside the gates of
 // shared experts), counting sort of the (token, choice) pairs by expert, and the fp32 residual update that gathers every
 // token's expert rows back in a fixed order (no atomics: a token's sum does not depend on the batch around it).
+#include <algorithm>
+
 #include "b200_serve.h"
 #include "common.cuh"
 #include "launch_count.h"
@@ -76,8 +78,8 @@ __device__ __forceinline__ void route_in_groups(float* z, float* pick, int n_out
 
 // one CTA per token: 16 warps compute the router outputs (fp32 dot over the width, eight loads in flight per lane),
 // thread 0 the softmax and the choice
-template <typename T>
-__global__ void __launch_bounds__(512) moe_route_kernel(const T* __restrict__ h, const float* __restrict__ wr,
+template <typename T, int MAX_THREADS = 512>
+__global__ void __launch_bounds__(MAX_THREADS) moe_route_kernel(const T* __restrict__ h, const float* __restrict__ wr,
                                                         const float* __restrict__ corr, const float* __restrict__ bias,
                                                         int on_logits, int width, int n_out, int top,
                                                         float scale, int groups, int keep, int* __restrict__ chosen,
@@ -295,12 +297,14 @@ extern "C" int b200_moe_route_sigmoid(const void* h, int h_dtype, const float* w
     cudaStream_t s = (cudaStream_t)stream;
     const size_t smem = ((size_t)2 * (n_out + n_gates) + width) * sizeof(float);
     if (smem > 48 * 1024) return B200_EUNSUPPORTED;
+    // a warp per output where 32 warps suffice; else rounds of equal length
+    const int n_all = n_out + n_gates, rounds = (n_all + 31) / 32, threads = 32 * std::max(4, (n_all + rounds - 1) / rounds);
     if (h_dtype == B200_BF16)
-        moe_route_kernel<__nv_bfloat16><<<n_tokens, 512, smem, s>>>((const __nv_bfloat16*)h, w_router, nullptr, nullptr, 0, width, n_out, top, 1.f,
-                                                                   0, 0, chosen, weight, 1, n_gates, gates);
+        moe_route_kernel<__nv_bfloat16, 1024><<<n_tokens, threads, smem, s>>>((const __nv_bfloat16*)h, w_router, nullptr, nullptr, 0, width, n_out, top,
+                                                                             1.f, 0, 0, chosen, weight, 1, n_gates, gates);
     else if (h_dtype == B200_F32)
-        moe_route_kernel<float><<<n_tokens, 512, smem, s>>>((const float*)h, w_router, nullptr, nullptr, 0, width, n_out, top, 1.f, 0, 0, chosen,
-                                                           weight, 1, n_gates, gates);
+        moe_route_kernel<float, 1024><<<n_tokens, threads, smem, s>>>((const float*)h, w_router, nullptr, nullptr, 0, width, n_out, top, 1.f, 0, 0,
+                                                                     chosen, weight, 1, n_gates, gates);
     else
         return B200_EINVAL;
     count_launch();

@@ -20,9 +20,19 @@ namespace b200 {
 // ---------------------------------------------------------------------------------------------------------------
 constexpr int kTileM = 64, kTileN = 64;
 
-template <int D, int DV, bool BLOCKS, bool BIAS>   // dim == D (a multiple of 32), vdim == DV (a multiple of 16); BLOCKS: a block mask or a window
+// the special-function unit's power of two (relative error 2^-22)
+__device__ __forceinline__ float pa_exp2(float x) {
+    float r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
+    return r;
+}
+
+enum { kNoBias = 0, kBias = 1, kBiasPadded = 2 };   // kBiasPadded: dim and vdim below the tile's
+
+template <int D, int DV, bool BLOCKS, int KIND>   // dim == D (a multiple of 32), vdim == DV (a multiple of 16); BLOCKS: a block mask or a window
 __global__ void __launch_bounds__(128, DV <= 128 ? 3 : 2) paged_attn_tile_kernel(const PA a) {
     using bf = __nv_bfloat16;
+    constexpr bool BIAS = KIND != kNoBias, PADDED = KIND == kBiasPadded;
     constexpr int RS = D + 8;                 // row stride in elements: 16-byte aligned, conflict-free fragment loads
     constexpr int CH = D / 8;                 // 16-byte chunks per row
     constexpr int RSV = DV + 8;               // the same for value rows
@@ -34,7 +44,7 @@ __global__ void __launch_bounds__(128, DV <= 128 ? 3 : 2) paged_attn_tile_kernel
     int* row_pos = reinterpret_cast<int*>(Vs + 2 * kTileN * RSV);   // [64], -1: no such row
     int* row_slot = row_pos + kTileM;
     float* bias_s = reinterpret_cast<float*>(row_slot + kTileM);       // BIAS: [2][128], entry 63 + (tile row - tile key)
-    const int dim = BIAS ? a.dim : D, vdim = BIAS ? a.vdim : DV;
+    const int dim = PADDED ? a.dim : D, vdim = PADDED ? a.vdim : DV;
     // the last rows of a prompt see the most keys: those tiles are scheduled first, the short ones fill the tail
     const int t0 = ((int)gridDim.x - 1 - (int)blockIdx.x) * kTileM, h = blockIdx.y;   // h: query unit (head, map)
     const int g = (h / a.maps) / (a.heads / a.kv_heads), ku = g * a.maps + h % a.maps;
@@ -49,7 +59,7 @@ __global__ void __launch_bounds__(128, DV <= 128 ? 3 : 2) paged_attn_tile_kernel
     for (int i = threadIdx.x; i < kTileM * CH; i += blockDim.x) {
         const int r = i / CH, c = i % CH;
         Pack16 v{{0u, 0u, 0u, 0u}};
-        if (r < rows && (!BIAS || c * 8 < dim)) v = ld16(Q + ((size_t)(t0 + r) * q_units + h) * dim + c * 8);
+        if (r < rows && (!PADDED || c * 8 < dim)) v = ld16(Q + ((size_t)(t0 + r) * q_units + h) * dim + c * 8);
         st16(Qs + r * RS + c * 8, v);
     }
     __syncthreads();
@@ -60,7 +70,7 @@ __global__ void __launch_bounds__(128, DV <= 128 ? 3 : 2) paged_attn_tile_kernel
     float o[DV / 8][4];
 #pragma unroll
     for (int nt = 0; nt < DV / 8; ++nt) o[nt][0] = o[nt][1] = o[nt][2] = o[nt][3] = 0.f;
-    const bool sig = a.sigmoid != 0;
+    const bool sig = !BIAS && a.sigmoid != 0;   // the host keeps sigmoid weights and caps away from the biased variants
     const float m0 = BIAS && a.sink ? a.sink[h / a.maps] : (a.denom_bias > 0.f || sig) ? 0.f : -1e30f, l0 = BIAS && a.sink ? 1.f : sig ? 1.f : a.denom_bias;
     const float* btab = BIAS && a.dist_bias ? a.dist_bias + (size_t)(h / a.maps) * a.dist_n : nullptr;
     const float far_bias = btab ? btab[a.dist_n - 1] : 0.f;
@@ -88,30 +98,34 @@ __global__ void __launch_bounds__(128, DV <= 128 ? 3 : 2) paged_attn_tile_kernel
         auto load_tile = [&](int k0, int buf) {
             bf* kd = Ks + buf * kTileN * RS;
             bf* vd = Vs + buf * kTileN * RSV;
-            // a thread brings chunk c of key row kr, and the DV / D value chunks that go with it (one page lookup for all)
             if constexpr (BIAS) {
-                constexpr int CHV = DV / 8, CHX = CH > CHV ? CH : CHV;
-                for (int i = threadIdx.x; i < kTileN * CHX; i += blockDim.x) {
-                    const int kr = i / CHX, c = i % CHX, j = k0 + kr;
-                    const bool ok = j < n_keys;
-                    const size_t row = ok ? (size_t)plist[j / a.page_rows] * a.page_rows + j % a.page_rows : 0;
-                    if (c < CH) {
-                        const bool in = ok && c * 8 < dim;
-                        const uint32_t kdst = (uint32_t)__cvta_generic_to_shared(kd + kr * RS + c * 8);
-                        asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(kdst), "l"(Kp + (in ? (row * k_units + ku) * dim + c * 8 : 0)), "r"(in ? 16u : 0u) : "memory");
-                    }
-                    if (c < CHV) {
-                        const bool in = ok && c * 8 < vdim;
-                        const uint32_t vdst = (uint32_t)__cvta_generic_to_shared(vd + kr * RSV + c * 8);
-                        asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(vdst), "l"(Vp + (in ? (row * a.kv_heads + g) * vdim + c * 8 : 0)), "r"(in ? 16u : 0u) : "memory");
-                    }
-                }
                 if (btab) {
                     const int dist = row_pos[seg] - seg - k0 + (int)threadIdx.x - 63;   // 128 threads, 127 distances
                     const uint32_t bdst = (uint32_t)__cvta_generic_to_shared(bias_s + buf * 128 + threadIdx.x);
                     asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(bdst), "l"(btab + min(max(dist, 0), a.dist_n - 1)) : "memory");
                 }
-            } else
+            }
+            if constexpr (PADDED || (DV % D != 0)) {
+                constexpr int CHV = DV / 8;
+                for (int i = threadIdx.x; i < kTileN * CH; i += blockDim.x) {
+                    const int kr = i / CH, c = i % CH, j = k0 + kr;
+                    const bool ok = j < n_keys;
+                    const size_t row = ok ? (size_t)plist[j / a.page_rows] * a.page_rows + j % a.page_rows : 0;
+                    const uint32_t bytes = (ok && c * 8 < dim) ? 16u : 0u;
+                    const int c0 = min(c * 8, dim - 8);
+                    const uint32_t kdst = (uint32_t)__cvta_generic_to_shared(kd + kr * RS + c * 8);
+                    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(kdst), "l"(Kp + (row * k_units + ku) * dim + c0), "r"(bytes) : "memory");
+                }
+                for (int i = threadIdx.x; i < kTileN * CHV; i += blockDim.x) {
+                    const int kr = i / CHV, c = i % CHV, j = k0 + kr;
+                    const bool ok = j < n_keys;
+                    const size_t row = ok ? (size_t)plist[j / a.page_rows] * a.page_rows + j % a.page_rows : 0;
+                    const uint32_t bytes = (ok && c * 8 < vdim) ? 16u : 0u;
+                    const int c0 = min(c * 8, vdim - 8);
+                    const uint32_t vdst = (uint32_t)__cvta_generic_to_shared(vd + kr * RSV + c * 8);
+                    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(vdst), "l"(Vp + (row * a.kv_heads + g) * vdim + c0), "r"(bytes) : "memory");
+                }
+            } else   // a thread brings chunk c of key row kr, and the DV / D value chunks that go with it (one page lookup for all)
             for (int i = threadIdx.x; i < kTileN * CH; i += blockDim.x) {
                 const int kr = i / CH, c = i % CH, j = k0 + kr;
                 const bool ok = j < n_keys;
@@ -125,6 +139,8 @@ __global__ void __launch_bounds__(128, DV <= 128 ? 3 : 2) paged_attn_tile_kernel
                     asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(vdst), "l"(Vp + (row * a.kv_heads + g) * DV + (c + e * CH) * 8), "r"(bytes) : "memory");
                 }
             }
+            __syncwarp();   // lanes that left the loops one after another commit together: a group closed by
+                            // part of a warp was seen not to cover the copies of the rest
             asm volatile("cp.async.commit_group;" ::: "memory");
         };
         __syncthreads();   // the buffers of the previous segment are no longer read
@@ -144,7 +160,7 @@ __global__ void __launch_bounds__(128, DV <= 128 ? 3 : 2) paged_attn_tile_kernel
             // K fragments of two k steps: matrices (k 0-7 | 8-15 | 16-23 | 24-31) of 8 keys
 #pragma unroll
             for (int ks = 0; ks < D / 16; ks += 2) {
-                if (BIAS && ks * 16 >= dim) continue;
+                if (PADDED && ks * 16 >= dim) continue;
                 uint32_t b4[kTileN / 8][4];
 #pragma unroll
                 for (int nt = 0; nt < kTileN / 8; ++nt)
@@ -163,7 +179,7 @@ __global__ void __launch_bounds__(128, DV <= 128 ? 3 : 2) paged_attn_tile_kernel
             // cap * tanh(v / cap): when every score of this thread's tile is small against the cap (the usual case) the odd
             // series x - x^3/3 + 2x^5/15 - 17x^7/315 is exact to fp32 rounding below |x| = 0.25 and costs no special-function
             // unit; otherwise (t - 1) / (t + 1) with t = e^(2x) (absolute error ~1e-7 * cap)
-            if (a.softcap > 0.f) {
+            if (!BIAS && a.softcap > 0.f) {
                 float big = 0.f;
 #pragma unroll
                 for (int nt = 0; nt < kTileN / 8; ++nt)
@@ -186,7 +202,7 @@ __global__ void __launch_bounds__(128, DV <= 128 ? 3 : 2) paged_attn_tile_kernel
                             s[nt][e] = a.softcap * __fdividef(t - 1.f, t + 1.f);
                         }
                 }
-            } else {
+            } else if (!BIAS || !btab) {
 #pragma unroll
                 for (int nt = 0; nt < kTileN / 8; ++nt)
 #pragma unroll
@@ -198,17 +214,23 @@ __global__ void __launch_bounds__(128, DV <= 128 ? 3 : 2) paged_attn_tile_kernel
 #pragma unroll
                         for (int nt = 0; nt < kTileN / 8; ++nt)
 #pragma unroll
-                            for (int e = 0; e < 4; ++e) s[nt][e] += far_bias;
+                            for (int e = 0; e < 4; ++e) s[nt][e] = fmaf(s[nt][e], sc_h, far_bias);
                     } else {
                         const float* bl = bias_s + buf * 128 + 63 + r_lo - tig * 2;
 #pragma unroll
                         for (int nt = 0; nt < kTileN / 8; ++nt)
 #pragma unroll
-                            for (int e = 0; e < 4; ++e) s[nt][e] += bl[(e & 2) * 4 - nt * 8 - (e & 1)];
+                            for (int e = 0; e < 4; ++e) s[nt][e] = fmaf(s[nt][e], sc_h, bl[(e & 2) * 4 - nt * 8 - (e & 1)]);
                     }
                 }
             }
             float mx[2] = {-INFINITY, -INFINITY};
+            if (BIAS && !BLOCKS && __all_sync(0xffffffffu, k0 + kTileN - 1 <= min(p_lo, p_hi))) {   // every row sees the whole tile
+#pragma unroll
+                for (int nt = 0; nt < kTileN / 8; ++nt)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) mx[e >> 1] = fmaxf(mx[e >> 1], s[nt][e]);
+            } else
 #pragma unroll
             for (int nt = 0; nt < kTileN / 8; ++nt)
 #pragma unroll
@@ -234,11 +256,14 @@ __global__ void __launch_bounds__(128, DV <= 128 ? 3 : 2) paged_attn_tile_kernel
                 m_run[hrow] = mn;
             }
             float sum[2] = {0.f, 0.f};
+            constexpr float kLog2E = 1.4426950408889634f;
+            const float ml[2] = {m_run[0] * kLog2E, m_run[1] * kLog2E};
 #pragma unroll
             for (int nt = 0; nt < kTileN / 8; ++nt)
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
-                    const float pv = __expf(s[nt][e] - m_run[e >> 1]);   // masked: exp(-inf) = 0
+                    // masked: exp(-inf) = 0
+                    const float pv = BIAS ? pa_exp2(fmaf(s[nt][e], kLog2E, -ml[e >> 1])) : __expf(s[nt][e] - m_run[e >> 1]);
                     s[nt][e] = pv;
                     sum[e >> 1] += pv;
                 }
@@ -260,7 +285,7 @@ __global__ void __launch_bounds__(128, DV <= 128 ? 3 : 2) paged_attn_tile_kernel
                 pf[3] = pa_pack(s[2 * kk + 1][2], s[2 * kk + 1][3]);
 #pragma unroll
                 for (int nt = 0; nt < DV / 8; nt += 2) {
-                    if (BIAS && nt * 8 >= vdim) continue;
+                    if (PADDED && nt * 8 >= vdim) continue;
                     // one transposed ldmatrix.x4: the V fragments of two column tiles
                     uint32_t b4[4];
                     pa_ldsm_x4_trans(b4, Vb + (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * RSV + (nt + (lane >> 4)) * 8);
@@ -281,32 +306,32 @@ __global__ void __launch_bounds__(128, DV <= 128 ? 3 : 2) paged_attn_tile_kernel
         if (a.out_f32) {
 #pragma unroll
             for (int nt = 0; nt < DV / 8; ++nt)
-                if (!BIAS || nt * 8 < vdim) *reinterpret_cast<float2*>(reinterpret_cast<float*>(a.out) + dst + nt * 8) = make_float2(o[nt][hrow * 2] * inv, o[nt][hrow * 2 + 1] * inv);
+                if (!PADDED || nt * 8 < vdim) *reinterpret_cast<float2*>(reinterpret_cast<float*>(a.out) + dst + nt * 8) = make_float2(o[nt][hrow * 2] * inv, o[nt][hrow * 2 + 1] * inv);
         } else {
 #pragma unroll
             for (int nt = 0; nt < DV / 8; ++nt)
-                if (!BIAS || nt * 8 < vdim) *reinterpret_cast<__nv_bfloat162*>(reinterpret_cast<bf*>(a.out) + dst + nt * 8) = __floats2bfloat162_rn(o[nt][hrow * 2] * inv, o[nt][hrow * 2 + 1] * inv);
+                if (!PADDED || nt * 8 < vdim) *reinterpret_cast<__nv_bfloat162*>(reinterpret_cast<bf*>(a.out) + dst + nt * 8) = __floats2bfloat162_rn(o[nt][hrow * 2] * inv, o[nt][hrow * 2 + 1] * inv);
         }
     }
 }
 
-template <int D, int DV, bool BIAS>
+template <int D, int DV, int KIND, bool MASKED = true>   // MASKED: the block-mask / window variant is built too
 static int launch_tile(const PA& a, cudaStream_t s) {
     static_assert(kTileM == kTileN, "the Q tile borrows a K buffer");
-    constexpr int smem = 2 * kTileN * (D + 8) * 2 + 2 * kTileN * (DV + 8) * 2 + 2 * kTileM * 4 + (BIAS ? 2 * 128 * 4 : 0);
+    constexpr int smem = 2 * kTileN * (D + 8) * 2 + 2 * kTileN * (DV + 8) * 2 + 2 * kTileM * 4 + (KIND != kNoBias ? 2 * 128 * 4 : 0);
     static unsigned long long done = 0;
-    static_assert(BIAS || DV % D == 0, "a thread brings DV / D value chunks with every key chunk");
+    static_assert(KIND != kNoBias || DV % D == 0, "a thread brings DV / D value chunks with every key chunk");
     const dim3 grid((a.n_tokens + kTileM - 1) / kTileM, a.heads * a.maps);
-    if (a.chunk > 0 || a.window > 0) {
+    if constexpr (MASKED) if (a.chunk > 0 || a.window > 0) {
         static unsigned long long done_b = 0;
-        const cudaError_t e = ensure_max_dynamic_smem((const void*)paged_attn_tile_kernel<D, DV, true, BIAS>, smem, done_b);
+        const cudaError_t e = ensure_max_dynamic_smem((const void*)paged_attn_tile_kernel<D, DV, true, KIND>, smem, done_b);
         if (e != cudaSuccess) return (int)e;
-        paged_attn_tile_kernel<D, DV, true, BIAS><<<grid, 128, smem, s>>>(a);
+        paged_attn_tile_kernel<D, DV, true, KIND><<<grid, 128, smem, s>>>(a);
         return (int)cudaGetLastError();
     }
-    const cudaError_t e = ensure_max_dynamic_smem((const void*)paged_attn_tile_kernel<D, DV, false, BIAS>, smem, done);
+    const cudaError_t e = ensure_max_dynamic_smem((const void*)paged_attn_tile_kernel<D, DV, false, KIND>, smem, done);
     if (e != cudaSuccess) return (int)e;
-    paged_attn_tile_kernel<D, DV, false, BIAS><<<grid, 128, smem, s>>>(a);
+    paged_attn_tile_kernel<D, DV, false, KIND><<<grid, 128, smem, s>>>(a);
     return (int)cudaGetLastError();
 }
 

@@ -251,6 +251,75 @@ __global__ void __launch_bounds__(kRowPrepThreads) qk_row_prepare_kernel(const Q
     }
 }
 
+// The same without rotation and bias for rows of at most 4 * PER * THREADS query and key columns in whole groups of four: the row, the
+// values and the weights are loaded up front and live in registers (one round trip to memory instead of two passes).
+template <typename T, int THREADS, int PER>
+__global__ void __launch_bounds__(THREADS) qk_row_prepare_reg_kernel(const QkPrep a) {
+    __shared__ float red[2][THREADS / 32];
+    const int t = blockIdx.x, nq = a.heads * a.dim, nk = a.kv_heads * a.dim, nv = a.v_heads * a.vdim, p = a.pos[t];
+    const float* row = a.proj + (size_t)t * a.ld_proj;
+    float4 v[PER], w[PER];
+    const float4 one = make_float4(1.f, 1.f, 1.f, 1.f);
+    float sq = 0.f, sk = 0.f;
+#pragma unroll
+    for (int k = 0; k < PER; ++k) {
+        const int i = 4 * (threadIdx.x + THREADS * k);
+        v[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+        w[k] = one;
+        if (i < nq + nk) {
+            v[k] = *reinterpret_cast<const float4*>(row + i);
+            const float* nw = i < nq ? a.q_norm : a.k_norm;
+            if (nw) w[k] = *reinterpret_cast<const float4*>(nw + (i < nq ? i : i - nq));
+        }
+    }
+    size_t cache_row = 0;
+    if (nk + nv > 0) cache_row = (size_t)a.pages[(size_t)a.slot[t] * a.max_pages + p / a.page_rows] * a.page_rows + p % a.page_rows;
+    for (int i = threadIdx.x * 4; i < nv; i += THREADS * 4) {
+        const float4 f = *reinterpret_cast<const float4*>(row + a.v_off + i);
+        const float vv[4] = {f.x, f.y, f.z, f.w};
+        prep_store<T, 4>(reinterpret_cast<T*>(a.v_pool) + cache_row * nv + i, vv);
+    }
+#pragma unroll
+    for (int k = 0; k < PER; ++k) {
+        const int i = 4 * (threadIdx.x + THREADS * k);
+        const float ss = v[k].x * v[k].x + v[k].y * v[k].y + v[k].z * v[k].z + v[k].w * v[k].w;
+        if (i < nq) sq += ss;
+        else sk += ss;
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+        sq += __shfl_xor_sync(0xffffffffu, sq, o);
+        sk += __shfl_xor_sync(0xffffffffu, sk, o);
+    }
+    if (threadIdx.x % 32 == 0) { red[0][threadIdx.x / 32] = sq; red[1][threadIdx.x / 32] = sk; }
+    const float mul = query_temp(a, p);
+    __syncthreads();
+    sq = sk = 0.f;
+#pragma unroll
+    for (int i = 0; i < THREADS / 32; ++i) { sq += red[0][i]; sk += red[1][i]; }
+    const float rq = a.q_norm ? 1.0f / sqrtf(sq / (float)nq + a.eps) : 1.f, rk = a.k_norm && nk > 0 ? 1.0f / sqrtf(sk / (float)nk + a.eps) : 1.f;
+    T* qd = reinterpret_cast<T*>(a.q_out) + (size_t)t * nq;
+    T* kd = reinterpret_cast<T*>(a.k_pool) + cache_row * nk;
+#pragma unroll
+    for (int k = 0; k < PER; ++k) {
+        const int i = 4 * (threadIdx.x + THREADS * k);
+        if (i >= nq + nk) continue;
+        const bool is_k = i >= nq;
+        const float r = is_k ? rk : rq, m = is_k ? 1.f : mul;
+        const float f[4] = {v[k].x * r * w[k].x * m, v[k].y * r * w[k].y * m, v[k].z * r * w[k].z * m, v[k].w * r * w[k].w * m};
+        prep_store<T, 4>(is_k ? kd + (i - nq) : qd + i, f);
+    }
+}
+template <typename T>
+static bool launch_row_prepare_reg(const QkPrep& a, int n_tokens, cudaStream_t s) {
+    const int quads = (a.heads + a.kv_heads) * a.dim / 4;
+    if (quads <= 256) qk_row_prepare_reg_kernel<T, 256, 1><<<n_tokens, 256, 0, s>>>(a);
+    else if (quads <= 1024) qk_row_prepare_reg_kernel<T, 512, 2><<<n_tokens, 512, 0, s>>>(a);
+    else if (quads <= 2048) qk_row_prepare_reg_kernel<T, 512, 4><<<n_tokens, 512, 0, s>>>(a);
+    else return false;
+    return true;
+}
+
 // Without convolution and head norm the preparation is a rotation and three scatters: a thread per four consecutive
 // dimensions of one head (or value head) of one token. It loads its own four values and, inside the rotated part, the
 // four of its rotate-half partner with 16-byte loads, and stores four values of the serving dtype at once.
@@ -363,7 +432,9 @@ extern "C" int b200_qk_prepare(const b200_qk_prepare_args* p, void* stream) {
         if (smem > 48 * 1024 - 128) return B200_EUNSUPPORTED;
         const bool vec = p->dim % 4 == 0 && p->ld_proj % 4 == 0 && al16(p->proj) && al16(p->q_out) && al16(p->k_pool) &&
                          (p->v_heads == 0 || (p->vdim % 4 == 0 && p->v_off % 4 == 0 && al16(p->v_pool)));
-        if (p->dtype == B200_BF16) {
+        const bool reg = vec && !p->rot_dims && !p->bias && (!p->q_norm || al16(p->q_norm)) && (!p->k_norm || al16(p->k_norm));
+        if (reg && (p->dtype == B200_BF16 ? launch_row_prepare_reg<__nv_bfloat16>(a, p->n_tokens, s) : p->dtype == B200_F32 && launch_row_prepare_reg<float>(a, p->n_tokens, s))) {
+        } else if (p->dtype == B200_BF16) {
             if (vec) qk_row_prepare_kernel<__nv_bfloat16, 4><<<p->n_tokens, kRowPrepThreads, smem, s>>>(a);
             else qk_row_prepare_kernel<__nv_bfloat16, 1><<<p->n_tokens, kRowPrepThreads, smem, s>>>(a);
         } else if (p->dtype == B200_F32) {

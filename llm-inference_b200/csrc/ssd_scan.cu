@@ -171,6 +171,7 @@ __device__ __forceinline__ void ssd_stage(float* dst, int stride, const float* s
     }
 }
 __device__ __forceinline__ void ssd_landed() {
+    __syncwarp();   // the lanes close their group of copies together
     asm volatile("cp.async.commit_group;\n\tcp.async.wait_group 0;" ::: "memory");
     __syncthreads();
 }

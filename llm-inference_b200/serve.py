@@ -613,3 +613,70 @@ def random_filipel(width, vocab, layers, seed=0):
                 w[p + "gate"], w[p + "up"], w[p + "down"] = rnd(f, width), rnd(f, width), rnd(width, f)
         cfg["layers"].append(dict(type=sp["type"], mixer=mx, mlp=ml))
     return cfg, w
+
+
+def random_mazotar(width, vocab, layers, streams=4, seed=0):
+    """(config, tensors) of a random Mazotar model. layers: dicts with type 'attention' (heads, kv_heads, dim, vdim, optionally
+    kv_from, buckets, bias_max) | 'mlstm' (heads, dim, vdim); ff = None | int (dense) | (ff, experts, top, shared_ff or None)"""
+    import math
+
+    import torch
+
+    g = torch.Generator().manual_seed(seed)
+
+    def rnd(*shape, s=None):
+        return (torch.randn(*shape, generator=g) * (s if s is not None else 1.0 / math.sqrt(shape[-1]))).to(torch.bfloat16)
+
+    cfg = dict(architecture="Mazotar", vocab=vocab, width=width, streams=streams, norm=dict(eps=1e-6), embedding=dict(scale=1.5), layers=[])
+    w = {"embed": rnd(vocab, width, s=1.0), "head": rnd(vocab, width), "final.norm": torch.ones(width)}
+
+    def sublayer(pre, q):
+        w[f"{pre}norm{q}"] = torch.ones(width)
+        w[f"{pre}hc{q}.in"] = torch.full((streams,), 1.0 / streams)
+        w[f"{pre}hc{q}.out"] = torch.ones(streams)
+        w[f"{pre}hc{q}.mix"] = 0.9 * torch.eye(streams) + 0.1 / streams
+
+    for i, sp in enumerate(layers):
+        pre, mp = f"l{i}.", f"l{i}.mix."
+        sublayer(pre, 1)
+        H, d, dv = sp["heads"], sp["dim"], sp["vdim"]
+        if sp["type"] == "mlstm":
+            mx = dict(heads=H, dim=d, vdim=dv, gate_cap=15.0)
+            for nm, rows in (("q", H * d), ("k", H * d), ("v", H * dv), ("g", H * dv), ("i", H), ("f", H)):
+                w[mp + nm] = rnd(rows, width)
+            w[mp + "i.b"], w[mp + "f.b"], w[mp + "norm"] = torch.zeros(H), torch.linspace(3.0, 6.0, H), torch.ones(H * dv)
+        else:
+            G = sp["kv_heads"]
+            mx = dict(heads=H, kv_heads=G, dim=d, vdim=dv, scale=1.0 / math.sqrt(d), bias_max=sp.get("bias_max", 1024),
+                      q_temp=dict(coef=0.1, every=1024))
+            w[mp + "q"], w[mp + "q.norm"] = rnd(H * d, width), torch.ones(H * d)
+            if sp.get("kv_from") is not None:
+                mx["kv_from"] = sp["kv_from"]
+            else:
+                w[mp + "k"], w[mp + "k.norm"], w[mp + "v"] = rnd(G * d, width), torch.ones(G * d), rnd(G * dv, width)
+            w[mp + "rel"], w[mp + "sink"] = rnd(sp.get("buckets", 32), H, s=0.5), torch.zeros(H)
+        w[mp + "o"] = rnd(width, H * dv)
+        ff = sp.get("ff")
+        if ff is None:
+            cfg["layers"].append(dict(type=sp["type"], mixer=mx, mlp=None))
+            continue
+        sublayer(pre, 2)
+        fp = pre + "mlp."
+
+        def unit(p, f):
+            w[p + "gate"], w[p + "up"], w[p + "down"] = rnd(f, width), rnd(f, width), rnd(width, f)
+        if isinstance(ff, int):
+            ml = dict(kind="dense", ff=ff)
+            unit(fp, ff)
+        else:
+            f, E, top, shared = ff
+            ml = dict(kind="moe", expert=dict(ff=f), router=dict(experts=E, top=top))
+            w[fp + "router"] = rnd(E, width)
+            for e in range(E):
+                unit(f"{fp}e{e}.", f)
+            if shared:
+                ml["shared"] = dict(ff=shared)
+                unit(fp + "shared.", shared)
+                w[fp + "shared.sg"] = rnd(1, width)
+        cfg["layers"].append(dict(type=sp["type"], mixer=mx, mlp=ml))
+    return cfg, w
