@@ -187,3 +187,96 @@ class Oracle:
 
     def forward(self, tokens, return_layers=False):
         return forward(self.cfg, self.w, tokens, keep_layers=return_layers)
+
+
+# ---------------------------------------------------------------------------------------------------------------
+# small random models for the tests (weights rounded to bfloat16, as a checkpoint stores them)
+# ---------------------------------------------------------------------------------------------------------------
+def random_model(seed, width, vocab, layers, streams=2, scale=1.5, eps=1e-5):
+    """layers: dicts with type 'attention' (heads, kv_heads, dim, vdim, buckets, bias_max, optionally scale, temp = (coef, every) or
+    None, kv_from, sharp) | 'mlstm' (heads, dim, vdim, cap); ff = None | int (dense) | (ff, experts, top, shared ff or None)."""
+    g = torch.Generator().manual_seed(seed)
+
+    def rnd(*shape, s=None):
+        return torch.randn(*shape, generator=g, dtype=torch.float32) * (s if s is not None else 1.0 / math.sqrt(shape[-1]))
+
+    cfg = dict(architecture="Mazotar", vocab=vocab, width=width, streams=streams, norm=dict(eps=eps), embedding=dict(scale=scale), layers=[])
+    w = {"embed": rnd(vocab, width, s=1.0), "head": rnd(vocab, width), "final.norm": 1 + rnd(width, s=0.1)}
+
+    def sublayer(pre, q):
+        w[f"{pre}norm{q}"] = 1 + rnd(width, s=0.2)
+        w[f"{pre}hc{q}.in"] = 0.6 + rnd(streams, s=0.4)
+        w[f"{pre}hc{q}.out"] = 1 + rnd(streams, s=0.5)
+        w[f"{pre}hc{q}.mix"] = 0.9 * torch.eye(streams) + rnd(streams, streams, s=0.3)
+
+    for i, sp in enumerate(layers):
+        pre = "l%d." % i
+        mp = pre + "mix."
+        sublayer(pre, 1)
+        H, d, dv = sp["heads"], sp["dim"], sp["vdim"]
+        if sp["type"] == "mlstm":
+            mx = dict(heads=H, dim=d, vdim=dv, gate_cap=sp.get("cap", 10.0))
+            for nm, rows in (("q", H * d), ("k", H * d), ("v", H * dv), ("g", H * dv)):
+                w[mp + nm] = rnd(rows, width)
+            w[mp + "i"], w[mp + "f"] = rnd(H, width, s=1.5 / math.sqrt(width)), rnd(H, width, s=1.5 / math.sqrt(width))
+            w[mp + "i.b"], w[mp + "f.b"], w[mp + "norm"] = rnd(H, s=1.0), 3 + rnd(H, s=1.5), 1 + rnd(H * dv, s=0.2)
+        else:
+            G = sp["kv_heads"]
+            mx = dict(heads=H, kv_heads=G, dim=d, vdim=dv, scale=sp.get("scale", 1.0 / math.sqrt(d)), bias_max=sp["bias_max"])
+            if sp.get("temp"):
+                mx["q_temp"] = dict(coef=sp["temp"][0], every=sp["temp"][1])
+            w[mp + "q"], w[mp + "q.norm"] = rnd(H * d, width), (1 + rnd(H * d, s=0.4)) * sp.get("sharp", 1.5)
+            if sp.get("kv_from") is not None:
+                mx["kv_from"] = sp["kv_from"]
+            else:
+                w[mp + "k"], w[mp + "k.norm"], w[mp + "v"] = rnd(G * d, width), 1 + rnd(G * d, s=0.4), rnd(G * dv, width)
+            w[mp + "rel"], w[mp + "sink"] = rnd(sp["buckets"], H, s=1.0), 1 + rnd(H, s=1.0)
+        w[mp + "o"] = rnd(width, H * dv)
+        ff = sp.get("ff")
+        if ff is None:
+            cfg["layers"].append(dict(type=sp["type"], mixer=mx, mlp=None))
+            continue
+        sublayer(pre, 2)
+        fp = pre + "mlp."
+
+        def unit(p, f):
+            w[p + "gate"], w[p + "up"], w[p + "down"] = rnd(f, width), rnd(f, width), rnd(width, f)
+        if isinstance(ff, int):
+            ml = dict(kind="dense", ff=ff)
+            unit(fp, ff)
+        else:
+            f, E, top, shared = ff
+            ml = dict(kind="moe", expert=dict(ff=f), router=dict(experts=E, top=top))
+            w[fp + "router"] = rnd(E, width, s=1.5 / math.sqrt(width))
+            for e in range(E):
+                unit(fp + "e%d." % e, f)
+            if shared:
+                ml["shared"] = dict(ff=shared)
+                unit(fp + "shared.", shared)
+                w[fp + "shared.sg"] = rnd(1, width, s=1.5 / math.sqrt(width))
+        cfg["layers"].append(dict(type=sp["type"], mixer=mx, mlp=ml))
+    return cfg, {k: v.to(torch.bfloat16).to(DT) for k, v in w.items()}
+
+
+def write_model(folder, cfg, w):
+    """config.json + model.safetensors with every tensor as bfloat16"""
+    import json
+    import os
+    import struct
+
+    os.makedirs(folder, exist_ok=True)
+    with open(os.path.join(folder, "config.json"), "w") as f:
+        json.dump(cfg, f)
+    header, blobs, off = {}, [], 0
+    for name, t in w.items():
+        raw = t.to(torch.bfloat16).contiguous().view(torch.int16).numpy().tobytes()
+        header[name] = dict(dtype="BF16", shape=list(t.shape), data_offsets=[off, off + len(raw)])
+        blobs.append(raw)
+        off += len(raw)
+    hj = json.dumps(header).encode()
+    hj += b" " * (-len(hj) % 8)
+    with open(os.path.join(folder, "model.safetensors"), "wb") as f:
+        f.write(struct.pack("<Q", len(hj)))
+        f.write(hj)
+        for b in blobs:
+            f.write(b)

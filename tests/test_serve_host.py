@@ -19,7 +19,7 @@ def S(pkg):
 
 def test_registry_lists_the_families(S):
     fams = S.lib().b200_model_families().decode().split(",")
-    assert "Nekodra" in fams and "Musilorn" in fams and "Tomalix" in fams and "Sakevik" in fams and "Filipel" in fams and "llama" in fams
+    assert "Nekodra" in fams and "Musilorn" in fams and "Tomalix" in fams and "Sakevik" in fams and "Filipel" in fams and "Mazotar" in fams and "llama" in fams
 
 
 def test_unknown_architecture_and_broken_config(S, tmp_path):
@@ -389,3 +389,94 @@ def test_filipel_oracle_pieces_agree_with_closed_forms():
     assert chosen.tolist() == [[0, 2]] and w[0].tolist() == pytest.approx([8 / 15, 7 / 15])
     gn = K.gated_group_norm(torch.ones(1, 4, dtype=D), torch.tensor([[1.0, 1.0, 5.0, 5.0]], dtype=D), torch.tensor([1.0, 2.0, 3.0, 4.0], dtype=D), 2, 0.0)
     assert torch.allclose(gn, torch.tensor([[1.0, 2.0, 3.0, 4.0]], dtype=D))
+
+
+def test_mazotar_configuration_errors_end_before_any_cuda_call(S, tmp_path):
+    import json
+    att = dict(type="attention", mixer=dict(heads=4, kv_heads=2, dim=4, vdim=6, scale=0.5, bias_max=30, q_temp=dict(coef=0.1, every=8)), mlp=None)
+    mem = dict(type="mlstm", mixer=dict(heads=2, dim=4, vdim=6, gate_cap=9.0), mlp=None)
+    moe = dict(kind="moe", expert=dict(ff=8), router=dict(experts=6, top=2), shared=dict(ff=4))
+
+    def refused(layers, text, **top):
+        cfg = dict(dict(architecture="Mazotar", width=8, vocab=5, streams=2, norm=dict(eps=1e-5), embedding=dict(scale=1.0), layers=layers), **top)
+        (tmp_path / "config.json").write_text(json.dumps(cfg))
+        with pytest.raises(RuntimeError, match=text):
+            S.Model(tmp_path)
+
+    def mixer(base, **kw):
+        return dict(base, mixer=dict(base["mixer"], **kw))
+    refused([], "required")
+    refused([att], "streams must be positive", streams=0)
+    refused([att], "16 streams", streams=17)
+    refused([dict(att, type="retention")], "not part of this family")
+    refused([dict(att, mixer=None)], "no mixer")
+    refused([dict(att, mlp=dict(kind="glu", ff=8))], "feed-forward kind")
+    refused([dict(mem, mlp=dict(kind="dense"))], "mlp.ff")
+    refused([dict(mem, mlp=dict(moe, shared=dict()))], "mlp.shared.ff")
+    refused([dict(mem, mlp=dict(moe, router=dict(experts=6, top=7)))], "router.top")
+    refused([dict(mem, mlp=dict(moe, router=dict(experts=60, top=17)))], "16 experts")
+    refused([mixer(att, bias_max=0)], "bias_max")
+    refused([mixer(att, heads=3)], "multiple of kv_heads")
+    refused([mixer(att, vdim=257)], "above 256")
+    refused([mixer(att, q_temp=dict(coef=0.1, every=0))], "q_temp.every")
+    refused([att, mixer(att, kv_from=1)], "kv_from")
+    refused([mem, mixer(att, kv_from=0)], "kv_from")
+    refused([att, mixer(att, kv_from=0), mixer(att, kv_from=1)], "kv_from")
+    refused([att, mixer(att, kv_from=0, vdim=5)], "kv_from: kv_heads, dim and vdim")
+    refused([mixer(mem, gate_cap=0.0)], "gate_cap")
+    refused([mixer(mem, dim=513)], "above 512")
+
+
+def test_mazotar_random_checkpoint_and_workspaces(S, tmp_path):
+    """the random checkpoint names what the loader asks for, and the workspace sizes follow the shape of the step"""
+    import json
+    att = dict(type="attention", heads=4, kv_heads=2, dim=8, vdim=8, buckets=6, bias_max=40)
+    cfg, w = S.random_mazotar(32, 50, [dict(type="mlstm", heads=2, dim=4, vdim=6, ff=24), dict(att, ff=(8, 4, 2, 16)), dict(att, kv_from=1, ff=None)], streams=3)
+    S.write_checkpoint(tmp_path, cfg, w)
+    raw = (tmp_path / "model.safetensors").read_bytes()
+    header = json.loads(raw[8:8 + int.from_bytes(raw[:8], "little")])
+    assert header["l0.mix.i.b"]["shape"] == [2] and header["l0.mix.norm"]["shape"] == [12] and header["l1.mix.rel"]["shape"] == [6, 4]
+    assert "l1.mix.k.norm" in header and "l2.mix.k" not in header and "l2.mix.k.norm" not in header and "l2.hc2.in" not in header
+    assert header["l1.hc2.mix"]["shape"] == [3, 3] and header["l1.mlp.shared.sg"]["shape"] == [1, 32] and header["l1.mlp.e3.down"]["shape"] == [32, 8]
+    L = S.lib()
+    assert L.b200_mlstm_norm_floats(8, 32) == 12 and L.b200_mlstm_norm_floats(9, 130) == 3 * 16     # n, padding, the maximum; a copy per 64 columns
+    assert L.b200_mlstm_workspace_bytes(127, 1, 4, 16, 8) == 0 and L.b200_mlstm_workspace_bytes(1000, 1, 4, 300, 8) == 0
+    assert L.b200_mlstm_workspace_bytes(128, 2, 4, 16, 8) >= 5 * 4 * (16 * 8 + 16 + 64 * 64 + 64) * 4
+
+
+def test_mazotar_oracle_pieces_agree_with_closed_forms():
+    """the plain implementation of the sixth family: sinusoids, buckets, the sink, the temperature, the memory against its unrolled
+    sum, the streams"""
+    import mazotar_oracle as K
+    g = torch.Generator().manual_seed(3)
+    D = torch.float64
+    s = K.sinusoids(4, 5)
+    assert s[0].tolist() == [0.0, 1.0, 0.0, 1.0, 0.0] and float(s[3, 2]) == pytest.approx(math.sin(3 * 10000 ** (-2 / 5)))
+    assert float(s[3, 3]) == pytest.approx(math.cos(3 * 10000 ** (-2 / 5)))
+    assert [K.bucket(n, 8, 64) for n in (0, 3, 4, 7, 8, 15, 16, 31, 32, 63, 64, 9999)] == [0, 3, 4, 4, 5, 5, 6, 6, 7, 7, 7, 7]
+    b = K.distance_bias(6, torch.tensor([[1.0, 10.0], [2.0, 20.0], [3.0, 30.0], [4.0, 40.0]], dtype=D), 8)
+    assert b[0, 5].tolist() == [4.0, 4.0, 3.0, 3.0, 2.0, 1.0] and b[1, 2].tolist() == [30.0, 20.0, 10.0, 0.0, 0.0, 0.0]
+    assert K.temperature(4, 0.5, 2).tolist() == pytest.approx([1.0, 1 + 0.5 * math.log(2), 1 + 0.5 * math.log(2), 1 + 0.5 * math.log(3)])
+    p = K.sink_softmax(torch.log(torch.tensor([[[1.0, 3.0]]], dtype=D)), torch.log(torch.tensor([4.0], dtype=D)))
+    assert p[0, 0].tolist() == pytest.approx([1 / 8, 3 / 8])
+    # zero queries: the weights are exp(bias) over their sum and the sink
+    v = torch.tensor([[[1.0]], [[5.0]]], dtype=D)
+    o = K.attend(torch.zeros(2, 1, 1, dtype=D), torch.ones(2, 1, 1, dtype=D), v, 1.0, torch.log(torch.tensor([[[2.0, 1.0], [6.0, 2.0]]], dtype=D)), torch.zeros(1, dtype=D))
+    assert o[:, 0, 0].tolist() == pytest.approx([2 / 3, (6 * 1 + 2 * 5) / 9])
+    # one head: the memory is a sum over older tokens; with the maximum taken out the floor of the denominator is 1
+    q, k, x, i = (torch.rand(5, generator=g, dtype=D) for _ in range(4))
+    f = -torch.rand(5, generator=g, dtype=D)
+    i = i * 3 - 1
+    y = K.mlstm_memory(q.view(5, 1, 1), k.view(5, 1, 1), x.view(5, 1, 1), i.view(5, 1), f.view(5, 1))
+    m = 0.0
+    for t in range(5):
+        m = max(float(f[t]) + m, float(i[t]))
+        wts = [math.exp(float(i[j] + f[j + 1:t + 1].sum())) for j in range(t + 1)]
+        num, den = sum(w_ * k[j] * x[j] for j, w_ in enumerate(wts)) * q[t], abs(sum(w_ * k[j] for j, w_ in enumerate(wts)) * q[t])
+        assert float(y[t, 0, 0]) == pytest.approx(float(num / (max(den, 1.0) + 1e-6 * math.exp(m))))
+    assert float(K.capped(torch.tensor(100.0, dtype=D), 7.0)) == pytest.approx(7.0)
+    chosen, w = K.route(torch.tensor([[0.0, math.log(3.0), -1.0]], dtype=D), 2)
+    assert chosen.tolist() == [[1, 0]] and w[0].tolist() == pytest.approx([0.75, 0.5])
+    W = {"in": torch.tensor([1.0, 2.0], dtype=D), "mix": torch.tensor([[1.0, 3.0], [0.0, 1.0]], dtype=D), "out": torch.tensor([1.0, -1.0], dtype=D)}
+    n = K.hyper(torch.tensor([[[3.0]], [[-1.0]]], dtype=D), W, "", torch.tensor([2.0], dtype=D), 0.0, lambda h: h * 5)
+    assert n[:, 0, 0].tolist() == [3.0 + 10.0, 3.0 * 3 - 1 - 10.0]     # u = 1, normed and weighted to 2, y = 10
