@@ -16,8 +16,10 @@
 //     mlstm_chain_kernel  the maximum at every chunk's start and the two factors of its carry;
 //     mlstm_carry_kernel  S and n at the start of every chunk, and what the entry leaves behind;
 //     mlstm_out_kernel    o_i = (exp(m - g_i) S^T q_i + exp(A_i - g_i) sum_j M_ij v_j) / denominator.
-//   Products run on tf32 tensor-core tiles (mma.sync m16n8k8) with fp32 accumulation; gates, maxima, factors, states, normalisers
-//   and everything between chunks are fp32, F and a are kept in double (differences of two large sums are exponentiated).
+//   Products run on tf32 tensor-core tiles (mma.sync m16n8k8) with fp32 accumulation. q, k and v, which are projections, enter as one
+//   tf32 number; what the recurrence itself made (the state, the weighted values, the weights M) enters as a sum of two, so it keeps
+//   21 bits. Gates, maxima, factors, states, normalisers and everything between chunks are fp32, F and a are kept in double
+//   (differences of two large sums are exponentiated).
 #include <cuda_bf16.h>
 #include <math.h>
 #include <stdlib.h>
@@ -171,6 +173,12 @@ __device__ __forceinline__ void ml_mma(float (&d)[4], const float (&a)[4], float
           "r"(__float_as_uint(b0)), "r"(__float_as_uint(b1)));
 }
 
+// v as the sum of two tf32 numbers
+__device__ __forceinline__ void ml_split(float v, float& hi, float& lo) {
+    hi = ml_tf32(v);
+    lo = ml_tf32(v - hi);
+}
+
 // F, a and A of a chunk (double) by warp 0, two tokens per lane; places beyond the chunk hold the last F and A and a = -inf
 struct MlGates {
     double F[kMlChunk], a[kMlChunk], A[kMlChunk];
@@ -317,7 +325,7 @@ __global__ void __launch_bounds__(128) mlstm_state_kernel(const ML a) {
         float4* v4 = reinterpret_cast<float4*>(Vs + (i / (kMlCols / 4)) * kMlVs) + i % (kMlCols / 4);
         const float w = wts[i / (kMlCols / 4)];
         const float4 v = *v4;
-        *v4 = make_float4(ml_tf32(v.x * w), ml_tf32(v.y * w), ml_tf32(v.z * w), ml_tf32(v.w * w));
+        *v4 = make_float4(v.x * w, v.y * w, v.z * w, v.w * w);
     }
     const size_t at = (size_t)ck.place * a.heads + h;
     if (p0 == 0)   // the normaliser's share of the chunk, fp32
@@ -340,7 +348,13 @@ __global__ void __launch_bounds__(128) mlstm_state_kernel(const ML a) {
             const float av[4] = {ml_tf32(ar[0]), ml_tf32(ar[8]), ml_tf32(ar[4 * st]), ml_tf32(ar[4 * st + 8])};
             const float* br = Vs + (k0 + tig) * kMlVs + gid;
 #pragma unroll
-            for (int nt = 0; nt < 8; ++nt) ml_mma(acc[nt], av, br[nt * 8], br[4 * kMlVs + nt * 8]);
+            for (int nt = 0; nt < 8; ++nt) {
+                float h0, l0, h1, l1;
+                ml_split(br[nt * 8], h0, l0);
+                ml_split(br[4 * kMlVs + nt * 8], h1, l1);
+                ml_mma(acc[nt], av, h0, h1);
+                ml_mma(acc[nt], av, l0, l1);
+            }
         }
 #pragma unroll
         for (int nt = 0; nt < 8; ++nt)
@@ -480,7 +494,7 @@ __global__ void __launch_bounds__(256) mlstm_out_kernel(const ML a) {
 #pragma unroll 4
     for (int i = threadIdx.x; i < kMlChunk * kMlChunk; i += 256) {
         float* v = Ms + (i / kMlChunk) * kMlMs + i % kMlChunk;
-        *v = ml_tf32(*v * r_new[i / kMlChunk]);
+        *v *= r_new[i / kMlChunk];
     }
     __syncthreads();
     const int warp = threadIdx.x / 32, lane = threadIdx.x % 32, gid = lane >> 2, tig = lane & 3;
@@ -493,17 +507,31 @@ __global__ void __launch_bounds__(256) mlstm_out_kernel(const ML a) {
         const float av[4] = {ml_tf32(ar[0]), ml_tf32(ar[8 * st]), ml_tf32(ar[4]), ml_tf32(ar[8 * st + 4])};
         const float* br = Ss + (k0 + tig) * kMlVs + q0 + gid;
 #pragma unroll
-        for (int nt = 0; nt < 4; ++nt) ml_mma(acc[nt], av, ml_tf32(br[nt * 8]), ml_tf32(br[4 * kMlVs + nt * 8]));
+        for (int nt = 0; nt < 4; ++nt) {
+            float h0, l0, h1, l1;
+            ml_split(br[nt * 8], h0, l0);
+            ml_split(br[4 * kMlVs + nt * 8], h1, l1);
+            ml_mma(acc[nt], av, h0, h1);
+            ml_mma(acc[nt], av, l0, l1);
+        }
     }
     const float e_lo = r_old[m0 + gid], e_hi = r_old[m0 + gid + 8];
 #pragma unroll
     for (int nt = 0; nt < 4; ++nt) { acc[nt][0] *= e_lo; acc[nt][1] *= e_lo; acc[nt][2] *= e_hi; acc[nt][3] *= e_hi; }
     for (int k0 = 0; k0 < m0 + 16; k0 += 8) {   // this chunk's own tokens, up to the warp's last row
         const float* ar = Ms + (m0 + gid) * kMlMs + k0 + tig;
-        const float av[4] = {ar[0], ar[8 * kMlMs], ar[4], ar[8 * kMlMs + 4]};   // rounded above
+        float ah[4], al[4];
+        ml_split(ar[0], ah[0], al[0]);
+        ml_split(ar[8 * kMlMs], ah[1], al[1]);
+        ml_split(ar[4], ah[2], al[2]);
+        ml_split(ar[8 * kMlMs + 4], ah[3], al[3]);
         const float* br = Vs + (k0 + tig) * kMlVs + q0 + gid;
 #pragma unroll
-        for (int nt = 0; nt < 4; ++nt) ml_mma(acc[nt], av, ml_tf32(br[nt * 8]), ml_tf32(br[4 * kMlVs + nt * 8]));
+        for (int nt = 0; nt < 4; ++nt) {
+            const float b0 = ml_tf32(br[nt * 8]), b1 = ml_tf32(br[4 * kMlVs + nt * 8]);
+            ml_mma(acc[nt], ah, b0, b1);
+            ml_mma(acc[nt], al, b0, b1);
+        }
     }
 #pragma unroll
     for (int nt = 0; nt < 4; ++nt)
