@@ -95,9 +95,12 @@ __global__ void __launch_bounds__(128, DV <= 128 ? 3 : 2) paged_attn_tile_kernel
         const int w_first = max(seg, warp * 16), w_last = min(seg_end, warp * 16 + 16) - 1;
         const int warp_keys = w_last >= w_first ? row_pos[w_last] + 1 : 0;
         const int warp_first = (BLOCKS && w_last >= w_first) ? pa_first_key(a, row_pos[w_first]) : 0;
+        const bool one_page = a.page_rows % kTileN == 0 && first_key % kTileN == 0;
         auto load_tile = [&](int k0, int buf) {
             bf* kd = Ks + buf * kTileN * RS;
             bf* vd = Vs + buf * kTileN * RSV;
+            // a tile that lies inside one page (the usual page sizes, walks from a tile's edge) takes one lookup
+            const size_t base = one_page ? (size_t)plist[k0 / a.page_rows] * a.page_rows + k0 % a.page_rows : 0;
             if constexpr (BIAS) {
                 if (btab) {
                     const int dist = row_pos[seg] - seg - k0 + (int)threadIdx.x - 63;   // 128 threads, 127 distances
@@ -110,7 +113,7 @@ __global__ void __launch_bounds__(128, DV <= 128 ? 3 : 2) paged_attn_tile_kernel
                 for (int i = threadIdx.x; i < kTileN * CH; i += blockDim.x) {
                     const int kr = i / CH, c = i % CH, j = k0 + kr;
                     const bool ok = j < n_keys;
-                    const size_t row = ok ? (size_t)plist[j / a.page_rows] * a.page_rows + j % a.page_rows : 0;
+                    const size_t row = one_page ? base + kr : ok ? (size_t)plist[j / a.page_rows] * a.page_rows + j % a.page_rows : 0;
                     const uint32_t bytes = (ok && c * 8 < dim) ? 16u : 0u;
                     const int c0 = min(c * 8, dim - 8);
                     const uint32_t kdst = (uint32_t)__cvta_generic_to_shared(kd + kr * RS + c * 8);
@@ -119,7 +122,7 @@ __global__ void __launch_bounds__(128, DV <= 128 ? 3 : 2) paged_attn_tile_kernel
                 for (int i = threadIdx.x; i < kTileN * CHV; i += blockDim.x) {
                     const int kr = i / CHV, c = i % CHV, j = k0 + kr;
                     const bool ok = j < n_keys;
-                    const size_t row = ok ? (size_t)plist[j / a.page_rows] * a.page_rows + j % a.page_rows : 0;
+                    const size_t row = one_page ? base + kr : ok ? (size_t)plist[j / a.page_rows] * a.page_rows + j % a.page_rows : 0;
                     const uint32_t bytes = (ok && c * 8 < vdim) ? 16u : 0u;
                     const int c0 = min(c * 8, vdim - 8);
                     const uint32_t vdst = (uint32_t)__cvta_generic_to_shared(vd + kr * RSV + c * 8);
@@ -129,7 +132,7 @@ __global__ void __launch_bounds__(128, DV <= 128 ? 3 : 2) paged_attn_tile_kernel
             for (int i = threadIdx.x; i < kTileN * CH; i += blockDim.x) {
                 const int kr = i / CH, c = i % CH, j = k0 + kr;
                 const bool ok = j < n_keys;
-                const size_t row = ok ? (size_t)plist[j / a.page_rows] * a.page_rows + j % a.page_rows : 0;
+                const size_t row = one_page ? base + kr : ok ? (size_t)plist[j / a.page_rows] * a.page_rows + j % a.page_rows : 0;
                 const uint32_t bytes = ok ? 16u : 0u;                 // beyond the sequence: zeros, nothing is read
                 const uint32_t kdst = (uint32_t)__cvta_generic_to_shared(kd + kr * RS + c * 8);
                 asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(kdst), "l"(Kp + (row * k_units + ku) * D + c * 8), "r"(bytes) : "memory");
