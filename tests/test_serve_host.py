@@ -480,3 +480,13 @@ def test_mazotar_oracle_pieces_agree_with_closed_forms():
     W = {"in": torch.tensor([1.0, 2.0], dtype=D), "mix": torch.tensor([[1.0, 3.0], [0.0, 1.0]], dtype=D), "out": torch.tensor([1.0, -1.0], dtype=D)}
     n = K.hyper(torch.tensor([[[3.0]], [[-1.0]]], dtype=D), W, "", torch.tensor([2.0], dtype=D), 0.0, lambda h: h * 5)
     assert n[:, 0, 0].tolist() == [3.0 + 10.0, 3.0 * 3 - 1 - 10.0]     # u = 1, normed and weighted to 2, y = 10
+
+
+def test_every_registered_family_has_a_program_of_its_own(S):
+    """bin/trace_run compiles one family's objects: the build has to know every family that the registry knows (llama is served by the
+    whole library)"""
+    import pathlib
+    import subprocess
+    pkg_dir = pathlib.Path(__file__).resolve().parent.parent / "llm-inference_b200"
+    known = subprocess.run(["make", "-s", "--no-print-directory", "-C", str(pkg_dir), "serve_families"], capture_output=True, text=True, check=True).stdout.split()
+    assert set(known) == set(S.lib().b200_model_families().decode().split(",")) - {"llama"}
